@@ -9,7 +9,7 @@ Against the reference (miniinfer/kvcache/kv_cache_manager.py, memory_pool.py):
   * page 0 of every pool is a dummy that padded tokens may write to (memory_pool.py:422-424);
   * a request keeps its slot and pages from admission to release, also between portions of its
     prompt (the reference frees the slot between chunks, llm_engine.py:1178-1181);
-  * pages behind a layer group's window are given back as soon as no later query can see them.
+  * pages behind a layer group's window or chunk are given back as soon as no later query can see them.
 
 The manager does no scheduling: callers ask ``can_append`` and then ``append``; ``commit`` makes
 the appended tokens part of the request after the step has run.
@@ -109,9 +109,7 @@ class PagedGroup:
 
   def first_needed_page(self, length: int) -> int:
     """Index of the first page that a query at position ``length`` (the next one) can still see."""
-    if self.spec.window is None:
-      return 0
-    return max(0, length - self.spec.window + 1) // self.page_size
+    return self.spec.first_needed(length) // self.page_size
 
   def sync(self) -> None:
     """Uploads the block-table rows that changed since the last call."""
@@ -167,7 +165,8 @@ class _Request:
 
 
 def pages_in_flight(window: int, page_size: int, max_step_tokens: int) -> int:
-  """The most pages a request holds in a group that keeps the last ``window`` positions: the window, what up to two
+  """The most pages a request holds in a group that keeps the last ``window`` positions (or the current chunk of that
+  many): the window, what up to two
   steps of ``max_step_tokens`` tokens add before the first of them is committed and the pages behind the window go
   back, and one page for where the window starts inside a page."""
   return -(-(window + 2 * max_step_tokens) // page_size) + 1
@@ -178,7 +177,7 @@ class KVCacheManager:
 
   ``num_pages`` is the size of a group that keeps every key.  A group that keeps a window needs no more than its
   requests can hold at a time: with ``max_step_tokens`` (the most tokens a request gets in one step) such a group
-  gets ``max_num_seqs * pages_in_flight(window, ...)`` pages, if that is less."""
+  gets ``max_num_seqs * pages_in_flight(window, ...)`` pages, if that is less.  So does a group that keeps a chunk."""
 
   def __init__(self, layer_specs: Sequence[Optional[CacheSpec]], page_size: int, num_pages: int,
                max_num_seqs: int, max_model_len: int, dtype: torch.dtype, device="cpu",
@@ -230,19 +229,19 @@ class KVCacheManager:
   @staticmethod
   def group_pages(spec: PagedKVSpec, page_size: int, num_pages: int, max_num_seqs: int, max_step_tokens: Optional[int]) -> int:
     """Pages of the group of ``spec`` when a group that keeps every key has ``num_pages``."""
-    if spec.window is None or max_step_tokens is None:
+    if spec.reach is None or max_step_tokens is None:
       return num_pages
-    return min(num_pages, max_num_seqs * (pages_in_flight(spec.window, page_size, max_step_tokens) + -(-spec.keep_first // page_size)))
+    return min(num_pages, max_num_seqs * (pages_in_flight(spec.reach, page_size, max_step_tokens) + -(-spec.keep_first // page_size)))
 
   @staticmethod
   def bytes_per_page(layer_specs: Sequence[Optional[CacheSpec]], page_size: int, dtype: torch.dtype,
                      windowed: Optional[bool] = None) -> int:
-    """Bytes that one more page costs in every paged group (``windowed`` None), in the groups that keep a window
+    """Bytes that one more page costs in every paged group (``windowed`` None), in the groups that keep a window or a chunk
     (True) or in those that keep every key (False)."""
     size = torch.empty((), dtype=dtype).element_size()
     total = 0
     for spec in flatten_specs(layer_specs):
-      if isinstance(spec, PagedKVSpec) and (windowed is None or windowed == (spec.window is not None)):
+      if isinstance(spec, PagedKVSpec) and (windowed is None or windowed == (spec.reach is not None)):
         total += 2 * spec.num_kv_heads * spec.head_dim * page_size * size
     return total
 
@@ -342,14 +341,14 @@ class KVCacheManager:
     r.reserved += n_new
 
   def commit(self, req_id: Hashable, n_new: int) -> None:
-    """The step has run: the tokens belong to the request.  Pages that a window has passed go back."""
+    """The step has run: the tokens belong to the request.  Pages that a window or a chunk has passed go back."""
     r = self._requests[req_id]
     if n_new > r.reserved:
       raise ValueError("commit of more tokens than were appended")
     r.reserved -= n_new
     r.length += n_new
     for g in self.paged_groups:
-      if g.spec.window is None:
+      if g.spec.reach is None:
         continue
       first = min(g.first_needed_page(r.length), len(r.pages[g.index]))
       dead = [i for i in range(g.kept_pages, first) if r.pages[g.index][i] != 0]

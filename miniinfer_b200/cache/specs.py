@@ -14,12 +14,14 @@ from typing import Optional, Tuple, Union
 @dataclass(frozen=True)
 class PagedKVSpec:
   """Keys and values of every position (``window is None``) or of the last ``window`` positions; with
-  ``keep_first`` the first positions of a request stay as well, whatever the window has passed."""
+  ``keep_first`` the first positions of a request stay as well, whatever the window has passed.  With ``chunk`` (and no
+  window) those of the chunk of that many positions, counted from position 0, which the next position lies in."""
 
   num_kv_heads: int
   head_dim: int
   window: Optional[int] = None
   keep_first: int = 0
+  chunk: Optional[int] = None
 
   def __post_init__(self):
     if self.num_kv_heads <= 0 or self.head_dim <= 0:
@@ -28,6 +30,19 @@ class PagedKVSpec:
       raise ValueError("window must be positive or None")
     if self.keep_first < 0:
       raise ValueError("keep_first must not be negative")
+    if self.chunk is not None and (self.chunk <= 0 or self.window is not None):
+      raise ValueError("chunk must be positive or None, and goes without a window")
+
+  @property
+  def reach(self) -> Optional[int]:
+    """The most positions a query looks back on (its own included), or None: all of them."""
+    return self.window if self.window is not None else self.chunk
+
+  def first_needed(self, length: int) -> int:
+    """The first position, kept first ones aside, that a query at position ``length`` (the next one) or later can see."""
+    if self.window is not None:
+      return max(0, length - self.window + 1)
+    return length // self.chunk * self.chunk if self.chunk is not None else 0
 
 
 @dataclass(frozen=True)

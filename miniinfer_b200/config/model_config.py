@@ -818,3 +818,142 @@ class LuporaxConfig(ModelConfig):
          "residual_mult": self.residual_mult, "logit_scale": self.logit_scale, "layers": [dict(x) for x in self.layers]}
     d.update(self.extra)
     return d
+
+
+@dataclass
+class ChunkedAttentionConfig:
+  """``layers[i].mixer`` of a Korurax ``attention`` layer: grouped-query attention inside chunks of ``mask.size`` positions (no
+  ``mask``: over every earlier token)."""
+
+  heads: int
+  kv_heads: int
+  dim: int
+  vdim: int
+  scale: float
+  chunk: Optional[int]
+
+
+@dataclass
+class ClampedDenseConfig:
+  """``layers[i].mlp`` of kind ``dense`` of a Korurax layer."""
+
+  ff: int
+  limit: float
+  kind: str = "dense"
+
+
+@dataclass
+class ScaledMoeConfig:
+  """``layers[i].mlp`` of kind ``moe`` of a Korurax layer: ``experts`` experts of width ``ff``, ``top`` of them a token, their
+  shares times ``scale``."""
+
+  ff: int
+  experts: int
+  top: int
+  scale: float
+  kind: str = "moe"
+
+
+@dataclass
+class KoruraxConfig(ModelConfig):
+  """Korurax: a decoder whose layers are listed one by one (``layers[i].{type, mixer, mlp}``), each a pre-norm layer whose
+  sublayers' outputs enter the stream times ``residual_mult`` and which hands on a weighted sum of all results so far; mixers of two
+  types - ``latent_attention`` and ``attention`` (chunked, with a distance bias, a sink and a gate per head); the feed-forward is
+  dense and clamped, a mixture of squared-ReLU experts, or absent.  The head is the embedding table, its logits capped at
+  ``logit_softcap``.  Other keys: ``architecture``, ``vocab``, ``width``, ``norm.eps``.  The design has no position limit of its own;
+  ``max_position_embeddings`` is only the engine's bound."""
+
+  architecture: str = "Korurax"
+  vocab: int = 0
+  width: int = 0
+  norm: Dict[str, Any] = field(default_factory=dict)
+  residual_mult: Any = None
+  logit_softcap: Any = None
+  layers: List[Dict[str, Any]] = field(default_factory=list)
+  max_position_embeddings: int = 1 << 30
+  initializer_range: float = 0.02
+
+  TYPES = ("latent_attention", "attention")
+
+  def validate(self) -> None:
+    if not self.architectures:
+      self.architectures = [self.architecture]
+    self.vocab_size = self.vocab
+    for key in ("vocab", "width"):
+      v = getattr(self, key)
+      if not isinstance(v, int) or isinstance(v, bool) or v <= 0:
+        raise ConfigError(f"{key} must be a positive integer, got {v!r}")
+    eps = self.norm.get("eps") if isinstance(self.norm, dict) else None
+    if not isinstance(eps, (int, float)) or isinstance(eps, bool) or not eps > 0:
+      raise ConfigError(f"norm.eps must be a positive number, got {eps!r}")
+    top = {"residual_mult": self.residual_mult, "logit_softcap": self.logit_softcap}
+    for key in top:
+      if not isinstance(top[key], (int, float)) or isinstance(top[key], bool):
+        raise ConfigError(f"{key} must be a number, got {top[key]!r}")
+    if not self.logit_softcap > 0:
+      raise ConfigError(f"logit_softcap must be positive, got {self.logit_softcap!r}")
+    if not self.layers:
+      raise ConfigError("layers must list at least one layer")
+    for i in range(len(self.layers)):
+      self.mixer_of(i)
+      self.mlp_of(i)
+
+  @property
+  def norm_eps(self) -> float:
+    return float(self.norm["eps"])
+
+  def type_of(self, i: int) -> str:
+    kind = self.layers[i].get("type")
+    if kind not in self.TYPES:
+      raise ConfigError(f"layers[{i}].type={kind!r} is not a mixer of this design (known: {', '.join(self.TYPES)})")
+    return kind
+
+  def mixer_of(self, i: int):
+    """The typed mixer configuration of layer ``i``: a ``LatentAttentionConfig`` or a ``ChunkedAttentionConfig``."""
+    kind = self.type_of(i)
+    m = self.layers[i].get("mixer")
+    where = f"layers[{i}].mixer"
+    if not isinstance(m, dict):
+      raise ConfigError(f"{where} is missing")
+    if kind == "latent_attention":
+      c = LatentAttentionConfig(*(_positive_int(m, k, where) for k in ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank")),
+                                _number(m, "scale", where), RotationConfig.read(m, where, ()))
+      if c.rot.dims != c.rot_dim:
+        raise ConfigError(f"{where}.rot.dims={c.rot.dims} must equal rot_dim={c.rot_dim}: the rotated part is rotated whole")
+      return c
+    mask = m.get("mask")
+    chunk = None
+    if mask is not None:
+      if not isinstance(mask, dict):
+        raise ConfigError(f"{where}.mask must be an object")
+      chunk = _positive_int(mask, "size", where + ".mask")
+    a = ChunkedAttentionConfig(*(_positive_int(m, k, where) for k in ("heads", "kv_heads", "dim", "vdim")), _number(m, "scale", where), chunk)
+    if a.heads % a.kv_heads:
+      raise ConfigError(f"{where}.heads={a.heads} must be a multiple of kv_heads={a.kv_heads}")
+    return a
+
+  def mlp_of(self, i: int):
+    """A ``ClampedDenseConfig``, a ``ScaledMoeConfig``, or None for a layer without a feed-forward."""
+    mlp = self.layers[i].get("mlp")
+    if mlp is None:
+      return None
+    where = f"layers[{i}].mlp"
+    kind = mlp.get("kind") if isinstance(mlp, dict) else mlp
+    if kind == "dense":
+      return ClampedDenseConfig(_positive_int(mlp, "ff", where), _number(mlp, "limit", where))
+    if kind != "moe":
+      raise ConfigError(f"{where}.kind={kind!r} is not known (dense, moe)")
+    expert, router = mlp.get("expert"), mlp.get("router")
+    if not isinstance(expert, dict) or not isinstance(router, dict):
+      raise ConfigError(f"{where} needs 'expert' and 'router'")
+    c = ScaledMoeConfig(_positive_int(expert, "ff", where + ".expert"), _positive_int(router, "experts", where + ".router"),
+                        _positive_int(router, "top", where + ".router"), _number(router, "scale", where + ".router"))
+    if c.top > c.experts:
+      raise ConfigError(f"{where}.router.top={c.top} is more than experts={c.experts}")
+    return c
+
+  def to_dict(self) -> Dict[str, Any]:
+    d = {"architecture": self.architecture, "vocab": self.vocab, "width": self.width, "norm": dict(self.norm),
+         "residual_mult": self.residual_mult, "logit_softcap": self.logit_softcap, "layers": [dict(x) for x in self.layers]}
+    d.update(self.extra)
+    return d

@@ -90,6 +90,33 @@ MI_API int mi_relu_squared(void* out, const void* x, int dtype, long long n, cud
   return 0;
 }
 
+namespace {
+__global__ void __launch_bounds__(256)
+softcap_kernel(float* __restrict__ x, size_t n, float cap) {
+  mi::grid_dependency_sync();
+  const float inv = 1.f / cap;
+  const size_t n4 = n / 4, step = (size_t)gridDim.x * blockDim.x;
+  const size_t i0 = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  float4* x4 = reinterpret_cast<float4*>(x);
+  for (size_t i = i0; i < n4; i += step) {
+    float4 v = x4[i];
+    v.x = cap * tanhf(v.x * inv); v.y = cap * tanhf(v.y * inv); v.z = cap * tanhf(v.z * inv); v.w = cap * tanhf(v.w * inv);
+    x4[i] = v;
+  }
+  for (size_t i = 4 * n4 + i0; i < n; i += step) x[i] = cap * tanhf(x[i] * inv);
+}
+}  // namespace
+
+// x <- cap * tanh(x / cap) over n float32 values, in place (a model's capped logits).
+MI_API int mi_softcap(float* x, long long n, float cap, cudaStream_t stream) {
+  MI_REQUIRE(n >= 0 && cap > 0.f && ((uintptr_t)x % 16) == 0, "softcap: bad size %lld, a cap that is not positive, or an unaligned buffer", n);
+  if (n == 0) return 0;
+  const size_t want = ((size_t)n / 4 + 256) / 256, most = (size_t)mi::sm_count() * 16;
+  mi::launch(softcap_kernel, dim3((unsigned)(want < most ? want : most)), dim3(256), 0, stream, x, (size_t)n, cap);
+  MI_LAUNCH_OK("softcap");
+  return 0;
+}
+
 // kind: a MiGlu; limit: the clamp of MI_GLU_CLAMPED.
 MI_API int mi_glu_mul(void* out, const void* gu, int dtype, int T, int I, int kind, float limit, cudaStream_t stream) {
   MI_REQUIRE(T >= 0 && I > 0, "glu_mul: bad sizes T=%d I=%d", T, I);

@@ -23,11 +23,12 @@
 //
 // Options (off when null): a sink per query head joins the denominator once, in the merge of the chunks
 // (exp(sink), unscaled, no value); an output gate multiplies the output row with sigmoid(gate[token,
-// head, :]); out_hd < head size writes only the first out_hd values of a head (padded cache rows).
+// head, :]), or with one gate per head; out_hd < head size writes only the first out_hd values of a head (padded cache rows).
 //
 // Shaped scores (attention_scores.cuh): a cap on the scaled scores, and sigmoid weights that are not normalised over the
 // keys - a score enters the online softmax as the logarithm of its weight, the pieces merge as ever, and the merged
-// output is multiplied with 2^m where the softmax divides by the sum.
+// output is multiplied with 2^m where the softmax divides by the sum; or a distance bias, which is taken off the scores of a
+// softmax.
 //
 // Compiled once per head size: -DMI_HEAD_DIM=<multiple of 16, 16..256>.
 #include "attention_scores.cuh"
@@ -97,6 +98,8 @@ struct DecodeArgs {
   int gate_stride, out_hd;
   float softcap;                 // shaped scores: the cap (0: none)
   const float* score_bias;       // [nh]: sigmoid weights; null: softmax
+  int gate_per_head;             // one gate per head, head h at h
+  const float* distance;         // [2, nh] r1, r2 of the distance bias; or null
 };
 
 // Gathers keys first .. first + BK of one kv head (K and V rows) into a stage; rows from `end` on are
@@ -143,7 +146,7 @@ decode_split_kernel(DecodeArgs a) {
   const int kvh = blockIdx.x, split = blockIdx.y, e = blockIdx.z;
   const int item = a.decode_items[e];
   const int p = a.ctx_len[item] - 1;                       // position of the query token
-  const int lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
+  const int lo = mi::first_visible(p, a.window);
   const int c0 = lo / a.chunk;
   // the request's first keep_first keys that the window has passed are pieces of their own, ahead of the window's
   const int kept = a.window > 0 ? min(a.keep_first, lo) : 0;
@@ -182,6 +185,16 @@ decode_split_kernel(DecodeArgs a) {
     const bool shaped = a.softcap > 0.f || a.score_bias != nullptr, sigmoid = a.score_bias != nullptr;
     const float row_bias[2] = {sigmoid && g < heads ? a.score_bias[kvh * G + g0 + g] : 0.f,
                                sigmoid && g + 8 < heads ? a.score_bias[kvh * G + g0 + g + 8] : 0.f};
+    const bool distance = a.distance != nullptr;
+    float row_r1[2] = {0.f, 0.f}, row_r2[2] = {0.f, 0.f};
+    if (distance) {
+#pragma unroll
+      for (int h = 0; h < 2; ++h)
+        if (g + 8 * h < heads) {
+          row_r1[h] = a.distance[kvh * G + g0 + g + 8 * h];
+          row_r2[h] = a.distance[a.nh + kvh * G + g0 + g + 8 * h];
+        }
+    }
     uint32_t qf[KSTEPS][4];
     float o[NT_O][4];
 #pragma unroll
@@ -228,8 +241,9 @@ decode_split_kernel(DecodeArgs a) {
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
           const int j = key0 + i * 8 + 2 * t + (c & 1);
-          const float v = j < k_end ? (shaped ? mi::shaped_logit2(s[i][c], a.scale, a.softcap, sigmoid, row_bias[c >> 1]) : s[i][c] * scale2)
+          float v = j < k_end ? (shaped ? mi::shaped_logit2(s[i][c], a.scale, a.softcap, sigmoid, row_bias[c >> 1]) : s[i][c] * scale2)
                                     : -INFINITY;
+          if (distance && j < k_end) v -= mi::distance_logit2(row_r1[c >> 1], row_r2[c >> 1], p - j);
           s[i][c] = v;
           mx[c >> 1] = fmaxf(mx[c >> 1], v);
         }
@@ -367,7 +381,7 @@ decode_split_kernel(DecodeArgs a) {
     }
     if (d < a.out_hd) {
       float y = acc * inv;
-      if (a.gate) y = __fdividef(y, 1.f + __expf(-__bfloat162float(a.gate[(size_t)row * a.gate_stride + (size_t)head * a.out_hd + d])));
+      if (a.gate) y = __fdividef(y, 1.f + __expf(-__bfloat162float(a.gate[(size_t)row * a.gate_stride + mi::gate_index(head, d, a.out_hd, a.gate_per_head)])));
       a.out[((size_t)row * a.nh + head) * a.out_hd + d] = __float2bfloat16_rn(y);
     }
   }
@@ -382,7 +396,7 @@ decode_merge_kernel(DecodeArgs a) {
   const int head = blockIdx.x, e = blockIdx.y;
   const int item = a.decode_items[e];
   const int p = a.ctx_len[item] - 1;
-  const int lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
+  const int lo = mi::first_visible(p, a.window);
   const int kept = a.window > 0 ? min(a.keep_first, lo) : 0;
   const int n_splits = (kept > 0 ? (kept - 1) / a.chunk + 1 : 0) + p / a.chunk - lo / a.chunk + 1;
   const int row = a.q_start[item];
@@ -401,7 +415,7 @@ decode_merge_kernel(DecodeArgs a) {
 #pragma unroll 8
     for (int s = 0; s < n_splits; ++s) acc = fmaf(po[(size_t)s * HD + d], exp2f(ml[2 * s] - m), acc);
     float y = acc * inv;
-    if (a.gate) y = __fdividef(y, 1.f + __expf(-__bfloat162float(a.gate[(size_t)row * a.gate_stride + (size_t)head * a.out_hd + d])));
+    if (a.gate) y = __fdividef(y, 1.f + __expf(-__bfloat162float(a.gate[(size_t)row * a.gate_stride + mi::gate_index(head, d, a.out_hd, a.gate_per_head)])));
     a.out[((size_t)row * a.nh + head) * a.out_hd + d] = __float2bfloat16_rn(y);
   }
 }
@@ -424,9 +438,10 @@ MI_API int mi_attention_decode_bf16(void* out, const void* q_base, int q_stride,
                                     int* counters, int n_dec, int nh, int nkv, int page_size, float scale,
                                     int window, int chunk, int max_splits, const float* sink, const void* gate,
                                     int gate_stride, int out_hd, int keep_first, float softcap, const float* score_bias,
-                                    cudaStream_t stream) {
+                                    int gate_per_head, const float* distance, cudaStream_t stream) {
   MI_REQUIRE(!(softcap < 0.f) && !(sink && score_bias), "attention_decode: softcap must not be negative, and sigmoid weights take no sink");
   MI_REQUIRE(out_hd > 0 && out_hd <= HD, "attention_decode: out_hd=%d must lie in 1..%d", out_hd, HD);
+  MI_REQUIRE(!(distance && score_bias), "attention_decode: a distance bias goes with a softmax");
   MI_REQUIRE(keep_first >= 0, "attention_decode: keep_first=%d must not be negative", keep_first);
   MI_REQUIRE(n_dec >= 0 && nh > 0 && nkv > 0 && nh % nkv == 0, "attention_decode: bad head counts nh=%d nkv=%d", nh, nkv);
   MI_REQUIRE(chunk >= BK && chunk <= MAX_CHUNK && chunk % BK == 0, "attention_decode: chunk=%d must be a multiple of %d up to %d", chunk, BK, MAX_CHUNK);
@@ -452,7 +467,7 @@ MI_API int mi_attention_decode_bf16(void* out, const void* q_base, int q_stride,
   a.nh = nh; a.nkv = nkv; a.page_size = page_size; a.window = window; a.chunk = chunk; a.max_splits = max_splits; a.keep_first = keep_first;
   a.scale = scale;
   a.sink = sink; a.gate = (const __nv_bfloat16*)gate; a.gate_stride = gate_stride; a.out_hd = out_hd;
-  a.softcap = softcap; a.score_bias = score_bias;
+  a.softcap = softcap; a.score_bias = score_bias; a.gate_per_head = gate_per_head; a.distance = distance;
   static bool configured = false;
   if (!configured) {
     cudaError_t err = cudaFuncSetAttribute(decode_split_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);

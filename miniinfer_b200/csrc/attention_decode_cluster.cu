@@ -89,6 +89,9 @@ struct ClusterArgs {
   const float* sink;               // [nh] or null: a logit per query head whose exponential joins the denominator once
   const __nv_bfloat16* gate;       // [T, gate_stride] or null: the output is multiplied with sigmoid(gate[row, head * HD + d])
   int gate_stride;
+  int gate_per_head;               // one gate per head, head h at h
+  float softcap;                   // shaped scores (attention_scores.cuh): a cap on the scores of a softmax (0: none)
+  const float* distance;           // [2, nh] r1, r2 of the distance bias; or null
 };
 
 // The last step of a head's output value: the sums A (weighted values) and L (weights) relative to the maximum M, the
@@ -102,10 +105,12 @@ __device__ __forceinline__ __nv_bfloat16 finish_value(const ClusterArgs& a, floa
     A = A * f;
   }
   float y = A / L;
-  if (a.gate) y = __fdividef(y, 1.f + __expf(-__bfloat162float(a.gate[(size_t)row * a.gate_stride + (size_t)head * HD + d])));
+  if (a.gate) y = __fdividef(y, 1.f + __expf(-__bfloat162float(a.gate[(size_t)row * a.gate_stride + mi::gate_index(head, d, HD, a.gate_per_head)])));
   return __float2bfloat16_rn(y);
 }
 
+// SHAPED: the form for capped scores and distance biases, compiled apart so that the plain softmax carries none of it.
+template <bool SHAPED>
 __global__ void __launch_bounds__(CTHREADS, 1)
 decode_cluster_kernel(const __grid_constant__ CUtensorMap kv_map, ClusterArgs a) {
   extern __shared__ __align__(1024) unsigned char smem_raw[];
@@ -142,7 +147,7 @@ decode_cluster_kernel(const __grid_constant__ CUtensorMap kv_map, ClusterArgs a)
   const int item = a.decode_items ? a.decode_items[e] : e;     // null: every item of the step brings one token, in order
   const int p = a.ctx_len[item] - 1;
   const int row = a.q_start[item];
-  const int lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
+  const int lo = mi::first_visible(p, a.window);
   const int j_first = lo / BK * BK;                              // first key of the request's first tile
   const int tiles = (p + 1 - j_first + BK - 1) / BK;
   const int per = (tiles + C - 1) / C;                           // tiles per block
@@ -296,12 +301,14 @@ decode_cluster_kernel(const __grid_constant__ CUtensorMap kv_map, ClusterArgs a)
 #pragma unroll
       for (int c = 0; c < 4; ++c) o[i][c] = 0.f;
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};   // heads 2t and 2t + 1
+    const TileScores shape = SHAPED ? tile_scores(a.scale, a.softcap, nullptr, a.distance, a.nh, kvh * G + 2 * t4, G - 2 * t4, p)
+                                    : plain_scores();
     for (int b = warp; b < nb; b += CW) {
       const int s = b % a.stages;
       mbar_wait(&full[s], (b / a.stages) & 1, abort, a.status);
       if (patch && b == nb - 1) mbar_wait(patched, 0, abort, a.status);
       const uint32_t kt = smem_u32(stage0 + (size_t)s * STAGE_BYTES);
-      consume_tile(kt, kt + TILE_BYTES, qf, o, m_run, l_run, j_first + (b0 + b) * BK, lo, p + 1, scale2, lane);
+      consume_tile(kt, kt + TILE_BYTES, qf, o, m_run, l_run, j_first + (b0 + b) * BK, lo, p + 1, scale2, lane, shape);
       __syncwarp();
       if (lane == 0) mbar_arrive(&empty[s]);
     }
@@ -414,8 +421,9 @@ MI_API int mi_attention_decode_cluster_fit(int cluster, int tiles_per_block) {
   if (stages < 1) return 0;
   const size_t smem = cluster_smem(stages, tiles_per_block);
   if (smem > 227 * 1024) return 0;
-  if (cudaFuncSetAttribute(decode_cluster_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) return 0;
-  if (cluster > 8 && cudaFuncSetAttribute(decode_cluster_kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) != cudaSuccess) {
+  // asked of the plain form; both forms hold one block an SM by their shared memory
+  if (cudaFuncSetAttribute(decode_cluster_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) return 0;
+  if (cluster > 8 && cudaFuncSetAttribute(decode_cluster_kernel<false>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) != cudaSuccess) {
     cudaGetLastError();
     return 0;
   }
@@ -431,7 +439,7 @@ MI_API int mi_attention_decode_cluster_fit(int cluster, int tiles_per_block) {
   cfg.attrs = attr;
   cfg.numAttrs = 1;
   int n = 0;
-  if (cudaOccupancyMaxActiveClusters(&n, decode_cluster_kernel, &cfg) != cudaSuccess) {
+  if (cudaOccupancyMaxActiveClusters(&n, decode_cluster_kernel<false>, &cfg) != cudaSuccess) {
     cudaGetLastError();
     return 0;
   }
@@ -444,7 +452,8 @@ int launch_cluster(void* out, const void* q_base, int q_stride, const void* kv_m
                    const int* ctx_len, const int* seq_slot, int* status, int n_dec, int nh, int nkv,
                    int page_size, float scale, int window, int cluster, int max_ctx_len, cudaStream_t stream,
                    int rope, const float* q_w, const float* k_w, const float* cos_sin, const int* slot_mapping, void* kv_layer, float eps,
-                   const float* sink = nullptr, const void* gate = nullptr, int gate_stride = 0) {
+                   const float* sink = nullptr, const void* gate = nullptr, int gate_stride = 0, int gate_per_head = 0, float softcap = 0.f,
+                   const float* distance = nullptr) {
   MI_REQUIRE(n_dec >= 0 && nh > 0 && nkv > 0 && nh % nkv == 0, "attention_decode_cluster: bad head counts nh=%d nkv=%d", nh, nkv);
   MI_REQUIRE(nh / nkv <= GP, "attention_decode_cluster: at most %d query heads per kv head (got %d)", GP, nh / nkv);
   MI_REQUIRE(cluster >= 1 && cluster <= 16, "attention_decode_cluster: cluster=%d is not in 1..16", cluster);
@@ -455,6 +464,7 @@ int launch_cluster(void* out, const void* q_base, int q_stride, const void* kv_m
   if (n_dec == 0) return 0;
   ClusterArgs a;
   a.sink = sink; a.gate = (const __nv_bfloat16*)gate; a.gate_stride = gate_stride;
+  a.gate_per_head = gate_per_head; a.softcap = softcap; a.distance = distance;
   a.out = (__nv_bfloat16*)out;
   a.q_base = (const __nv_bfloat16*)q_base;
   a.q_stride = q_stride;
@@ -471,7 +481,7 @@ int launch_cluster(void* out, const void* q_base, int q_stride, const void* kv_m
   a.kv_layer = (__nv_bfloat16*)kv_layer; a.eps = eps;
   MI_REQUIRE(!rope || HD == 128, "attention_decode_cluster: norm and rotation inside the kernel are for head size 128 (got %d)", HD);
   // the most tiles a request can have (a window may start anywhere in its first tile), and a block's share
-  const int span = window > 0 && window < max_ctx_len ? window : max_ctx_len;
+  const int span = mi::visible_span(max_ctx_len, window);
   const int tiles = (span + BK - 1) / BK + 1;
   a.max_tiles = (tiles + cluster - 1) / cluster;
   const int stages = cluster_stages(a.max_tiles);
@@ -479,14 +489,17 @@ int launch_cluster(void* out, const void* q_base, int q_stride, const void* kv_m
   a.stages = stages;
   const size_t smem = cluster_smem(stages, a.max_tiles);
   MI_REQUIRE(smem <= 227 * 1024, "attention_decode_cluster: shared memory does not suffice (%zu bytes)", smem);
-  static bool configured = false, wide = false;
+  const bool shaped = softcap > 0.f || distance != nullptr;
+  auto kernel = shaped ? decode_cluster_kernel<true> : decode_cluster_kernel<false>;
+  static bool configured_of[2] = {false, false}, wide_of[2] = {false, false};
+  bool &configured = configured_of[shaped], &wide = wide_of[shaped];
   if (!configured) {
-    cudaError_t err = cudaFuncSetAttribute(decode_cluster_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
     if (err != cudaSuccess) return mi_fail("attention_decode_cluster: cannot get shared memory: %s", cudaGetErrorString(err));
     configured = true;
   }
   if (cluster > 8 && !wide) {
-    cudaError_t err = cudaFuncSetAttribute(decode_cluster_kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+    cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
     if (err != cudaSuccess) return mi_fail("attention_decode_cluster: clusters of %d blocks are not available: %s", cluster, cudaGetErrorString(err));
     wide = true;
   }
@@ -513,7 +526,7 @@ int launch_cluster(void* out, const void* q_base, int q_stride, const void* kv_m
   }
   cfg.attrs = attr;
   cfg.numAttrs = na;
-  cudaError_t err = cudaLaunchKernelEx(&cfg, decode_cluster_kernel, map, a);
+  cudaError_t err = cudaLaunchKernelEx(&cfg, kernel, map, a);
   if (err != cudaSuccess) return mi_fail("attention_decode_cluster: launch failed: %s", cudaGetErrorString(err));
   return 0;
 }
@@ -524,10 +537,11 @@ MI_API int mi_attention_decode_cluster(void* out, const void* q_base, int q_stri
                                        const int* block_table, int bt_stride, const int* decode_items, const int* q_start,
                                        const int* ctx_len, const int* seq_slot, int* status, int n_dec, int nh, int nkv,
                                        int page_size, float scale, int window, int cluster, int max_ctx_len, cudaStream_t stream,
-                                       const float* sink, const void* gate, int gate_stride) {
+                                       const float* sink, const void* gate, int gate_stride, int gate_per_head, float softcap,
+                                       const float* distance) {
   return launch_cluster(out, q_base, q_stride, kv_map, block_table, bt_stride, decode_items, q_start, ctx_len, seq_slot, status, n_dec,
                         nh, nkv, page_size, scale, window, cluster, max_ctx_len, stream, 0, nullptr, nullptr, nullptr, nullptr, nullptr, 0.f,
-                        sink, gate, gate_stride);
+                        sink, gate, gate_stride, gate_per_head, softcap, distance);
 }
 
 // The same for a step of decode tokens only, with the step before attention inside (head size 128, the whole head
@@ -548,7 +562,8 @@ MI_API int mi_attention_decode_cluster_rope(void* out, const void* qkv, int q_st
 MI_API int mi_attention_decode_cluster_supported() { return 0; }
 MI_API int mi_attention_decode_cluster_fit(int, int) { return 0; }
 MI_API int mi_attention_decode_cluster(void*, const void*, int, const void*, const int*, int, const int*, const int*, const int*,
-                                       const int*, int*, int, int, int, int, float, int, int, int, cudaStream_t, const float*, const void*, int) {
+                                       const int*, int*, int, int, int, int, float, int, int, int, cudaStream_t, const float*, const void*, int, int, float,
+                                       const float*) {
   return mi_fail("attention_decode_cluster: head size %d has no such kernel", MI_HEAD_DIM);
 }
 MI_API int mi_attention_decode_cluster_rope(void*, const void*, int, const void*, const int*, int, const int*, const int*, const int*,

@@ -89,13 +89,34 @@ __device__ __forceinline__ uint32_t tile_addr(uint32_t tile, int r, int c) {
 // `jb`: the token of the tile's first row; qf: the query fragments (head lane / 4, dims 16k + 2(lane % 4) ..
 // and + 8); o[db][c]: dim db*16 + lane/4 + 8*(c/2), head 2(lane % 4) + (c & 1); m_run, l_run: heads
 // 2(lane % 4) and + 1, the sums still spread over the lanes that hold different keys.  `shape`: shaped scores
-// (attention_scores.cuh), with the biases of this thread's two heads.
+// (attention_scores.cuh), with the numbers of this thread's two heads; `pos`: the query's position (for a distance bias).
 struct TileScores {
-  bool shaped, sigmoid;
+  bool shaped, sigmoid, distance;
   float scale, softcap;
-  float bias[2];
+  float bias[2], r1[2], r2[2];
+  int pos;
 };
-__device__ __forceinline__ TileScores plain_scores() { return TileScores{false, false, 0.f, 0.f, {0.f, 0.f}}; }
+__device__ __forceinline__ TileScores plain_scores() {
+  return TileScores{false, false, false, 0.f, 0.f, {0.f, 0.f}, {0.f, 0.f}, {0.f, 0.f}, 0};
+}
+// The scores' shape for the heads head0 and head0 + 1 (of which `heads` exist) of a launch's options.
+__device__ __forceinline__ TileScores tile_scores(float scale, float softcap, const float* score_bias, const float* distance, int nh,
+                                                  int head0, int heads, int pos) {
+  TileScores s = plain_scores();
+  s.shaped = softcap > 0.f || score_bias != nullptr;
+  s.sigmoid = score_bias != nullptr;
+  s.distance = distance != nullptr;
+  s.scale = scale;
+  s.softcap = softcap;
+  s.pos = pos;
+#pragma unroll
+  for (int c = 0; c < 2; ++c)
+    if (c < heads) {
+      if (score_bias) s.bias[c] = score_bias[head0 + c];
+      if (distance) { s.r1[c] = distance[head0 + c]; s.r2[c] = distance[nh + head0 + c]; }
+    }
+  return s;
+}
 
 __device__ __forceinline__ void consume_tile(uint32_t kt, uint32_t vt, const uint32_t (&qf)[KSTEPS][2], float (&o)[HD / 16][4],
                                              float (&m_run)[2], float (&l_run)[2], int jb, int k_lo, int k_end, float scale2,
@@ -125,9 +146,10 @@ __device__ __forceinline__ void consume_tile(uint32_t kt, uint32_t vt, const uin
 #pragma unroll
     for (int c = 0; c < 4; ++c) {
       const int j = jb + i * 16 + g + 8 * (c >> 1);
-      const float v = (j >= k_lo && j < k_end)
+      float v = (j >= k_lo && j < k_end)
                           ? (shape.shaped ? mi::shaped_logit2(sc[i][c], shape.scale, shape.softcap, shape.sigmoid, shape.bias[c & 1]) : sc[i][c] * scale2)
                           : -INFINITY;
+      if (shape.distance && j >= k_lo && j < k_end) v -= mi::distance_logit2(shape.r1[c & 1], shape.r2[c & 1], shape.pos - j);
       sc[i][c] = v;
       mx[c & 1] = fmaxf(mx[c & 1], v);
     }

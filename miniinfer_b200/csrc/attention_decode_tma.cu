@@ -73,7 +73,7 @@ struct Item {                                // what the producer tells the cons
   int j0;                                    // first key of tile 0 (a multiple of 64)
   int k_lo, k_end;                           // keys that count: k_lo <= j < k_end
   int row;                                   // the request's row in the step
-  int pad;                                   // keeps the size a multiple of 8 bytes
+  int pos;                                   // the query's position  (ten ints: the size is a multiple of 8 bytes)
 };
 
 struct Args {
@@ -97,10 +97,12 @@ struct Args {
   int gate_stride;
   float softcap;                 // shaped scores (attention_scores.cuh): the cap (0: none)
   const float* score_bias;       // [nh]: sigmoid weights, nothing normalised over the keys; null: softmax
+  int gate_per_head;             // one gate per head, head h at h
+  const float* distance;         // [2, nh] r1, r2 of the distance bias; or null
 };
 
 __device__ __forceinline__ float gated(const Args& a, float y, int row, int head, int d) {
-  if (a.gate) y = __fdividef(y, 1.f + __expf(-__bfloat162float(a.gate[(size_t)row * a.gate_stride + (size_t)head * HD + d])));
+  if (a.gate) y = __fdividef(y, 1.f + __expf(-__bfloat162float(a.gate[(size_t)row * a.gate_stride + mi::gate_index(head, d, HD, a.gate_per_head)])));
   return y;
 }
 
@@ -157,7 +159,7 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map, Args a) {
       int v = 0;
       if (e < a.n_dec) {
         const int p = a.ctx_len[a.decode_items[e]] - 1;
-        const int lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
+        const int lo = mi::first_visible(p, a.window);
         v = (p + 1 - lo / BK * BK + BK - 1) / BK;
       }
       int x = v;
@@ -210,7 +212,7 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map, Args a) {
       const int b1 = (int)min((long long)nt, b0 + (t_end - t));
       const int item = a.decode_items[e];
       const int p = a.ctx_len[item] - 1;
-      const int lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
+      const int lo = mi::first_visible(p, a.window);
       const int j_first = lo / BK * BK;
       const int j0 = j_first + b0 * BK;
       const int nb = b1 - b0;
@@ -261,7 +263,7 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map, Args a) {
         mbar_wait(&qempty[qp], ((it / NI) & 1) ^ 1, abort, a.status);
         Item d;
         d.nb = nb; d.e = e; d.kvh = kvh; d.split = split; d.n_splits = n_splits;
-        d.j0 = j0; d.k_lo = k_lo; d.k_end = k_end; d.row = row;
+        d.j0 = j0; d.k_lo = k_lo; d.k_end = k_end; d.row = row; d.pos = p;
         items[qp] = d;
         // the query heads of this kv head are neighbours in the row: one copy
         mbar_expect_tx(&qfull[qp], (uint32_t)(G * HD * 2));
@@ -417,13 +419,7 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map, Args a) {
 #pragma unroll
         for (int c = 0; c < 4; ++c) o[i][c] = 0.f;
       float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};   // heads 2t and 2t + 1
-      TileScores shape = plain_scores();
-      if (a.softcap > 0.f || a.score_bias) {
-        shape.shaped = true; shape.sigmoid = a.score_bias != nullptr; shape.scale = a.scale; shape.softcap = a.softcap;
-#pragma unroll
-        for (int c = 0; c < 2; ++c)
-          shape.bias[c] = (a.score_bias && 2 * t4 + c < heads) ? a.score_bias[d.kvh * G + g0 + 2 * t4 + c] : 0.f;
-      }
+      const TileScores shape = tile_scores(a.scale, a.softcap, a.score_bias, a.distance, a.nh, d.kvh * G + g0 + 2 * t4, heads - 2 * t4, d.pos);
 
       // tile gb of this block's stream goes to warp gb mod 3 (it owns the stages gb mod `stages` can be);
       // `rank` is the warp's place among the item's tiles, which fixes the order of the merge
@@ -555,8 +551,9 @@ MI_API int mi_attention_decode_tma(void* out, const void* q_base, int q_stride, 
                                    const int* ctx_len, const int* seq_slot, float* scratch, int* counters, int* status,
                                    int n_dec, int nh, int nkv, int page_size, float scale, int window, int chunk,
                                    int max_splits, int num_sms, cudaStream_t stream, const float* sink, const void* gate, int gate_stride,
-                                   float softcap, const float* score_bias) {
+                                   float softcap, const float* score_bias, int gate_per_head, const float* distance) {
   MI_REQUIRE(!(softcap < 0.f) && !(sink && score_bias), "attention_decode_tma: softcap must not be negative, and sigmoid weights take no sink");
+  MI_REQUIRE(!(distance && score_bias), "attention_decode_tma: a distance bias goes with a softmax");
   MI_REQUIRE(n_dec >= 0 && nh > 0 && nkv > 0 && nh % nkv == 0, "attention_decode_tma: bad head counts nh=%d nkv=%d", nh, nkv);
   MI_REQUIRE(page_size % BK == 0, "attention_decode_tma: page_size=%d must be a multiple of %d", page_size, BK);
   MI_REQUIRE(chunk >= BK && chunk % BK == 0, "attention_decode_tma: chunk=%d must be a multiple of %d", chunk, BK);
@@ -585,7 +582,7 @@ MI_API int mi_attention_decode_tma(void* out, const void* q_base, int q_stride, 
   a.gp = G < 16 ? G : 16;
   a.scale = scale;
   a.sink = sink; a.gate = (const __nv_bfloat16*)gate; a.gate_stride = gate_stride;
-  a.softcap = softcap; a.score_bias = score_bias;
+  a.softcap = softcap; a.score_bias = score_bias; a.gate_per_head = gate_per_head; a.distance = distance;
   int stages = MAX_STAGES;
   while (stages > CONSUMERS && smem_bytes(stages, a.gp, max_splits, n_dec) > 220 * 1024) stages -= CONSUMERS;
   MI_REQUIRE(smem_bytes(stages, a.gp, max_splits, n_dec) <= 227 * 1024, "attention_decode_tma: shared memory does not suffice");

@@ -1,8 +1,9 @@
 // Attention over the paged cache for any mix of prompt portions and decode tokens, any head size
-// that is a multiple of 4 up to 256, any page size, float32 or bf16 storage, float32 arithmetic.
+// that is a multiple of 4 up to 640, any page size, float32 or bf16 storage, float32 arithmetic.
 //
 // One warp per (token, query head).  The warp walks the keys the token may see - positions
-// max(0, p - window + 1) .. p of its own request, p being the token's position - in chunks of 32
+// max(0, p - window + 1) .. p of its own request (or those of its chunk: first_visible, attention_scores.cuh), p being
+// the token's position - in chunks of 32
 // aligned to multiples of 32, with an online softmax.  The order of the arithmetic depends on
 // (p, window, keep_first) only, so the result for a token is bit-equal however the request was cut into steps
 // and whatever else is in the batch.  This is the attention of the 32-bit path, and the reference
@@ -18,19 +19,21 @@
 // Three options, all off when their pointers are null: a sink per query head - a learned logit whose
 // exponential joins the softmax's denominator once, unscaled, with no key and no value (the running
 // maximum starts at the sink and the running sum at 1); an output gate - the output row is multiplied
-// element by element with sigmoid(gate[token, head, :]); and out_hd < head_dim - only the first out_hd
+// element by element with sigmoid(gate[token, head, :]), or as a whole with the sigmoid of one gate per head; and out_hd < head_dim - only the first out_hd
 // values of a head are written (the cache rows are padded).  With a window, keep_first > 0 lets every token also see
 // the first keep_first keys of its request, at their true positions.
 //
 // Two more, for designs that shape the scores: softcap > 0 replaces a scaled score s by softcap * tanh(s / softcap) before
 // anything else sees it; and with score_bias (one float per query head) the weights are not a softmax at all - the weight
 // of a visible key is sigmoid(s + score_bias[head]), nothing is normalised over the keys, and the output is the plain sum
-// of the weighted values (a sink has no meaning then).
+// of the weighted values (a sink has no meaning then).  And for a softmax, distance: two floats per query head (all r1, then
+// all r2); a score loses r1 * ln(1 + r2 * (p - j)).
+#include "attention_scores.cuh"
 #include "common.cuh"
 
 namespace {
 
-constexpr int MAX_HD = 256;
+constexpr int MAX_HD = 640;
 constexpr int WARPS = 4;
 
 template <typename T>
@@ -65,16 +68,18 @@ __device__ __forceinline__ float dot_row<__nv_bfloat16>(const __nv_bfloat16* __r
   return s;
 }
 
-template <typename T>
+// HD_MAX: the largest head size the form takes (its output row lies in registers): 256, or 640 for latents wider than that.
+template <typename T, int HD_MAX>
 __global__ void __launch_bounds__(WARPS * 32)
 attention_generic_kernel(T* __restrict__ out, const T* __restrict__ q_base, int q_stride,
                          const T* __restrict__ kv_layer, const int* __restrict__ block_table, int bt_stride,
                          const int* __restrict__ token_item, const int* __restrict__ positions,
                          const int* __restrict__ seq_slot, int nh, int nkv, int hd, int page_size,
                          float scale, int window, const float* __restrict__ sink, const T* __restrict__ gate,
-                         int gate_stride, int out_hd, int keep_first, float softcap, const float* __restrict__ score_bias) {
+                         int gate_stride, int out_hd, int keep_first, float softcap, const float* __restrict__ score_bias,
+                         int gate_per_head, const float* __restrict__ distance) {
   mi::grid_dependency_sync();
-  __shared__ float qs[WARPS][MAX_HD];
+  __shared__ float qs[WARPS][HD_MAX];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int tkn = blockIdx.y;
   const int head = blockIdx.x * WARPS + warp;
@@ -83,7 +88,7 @@ attention_generic_kernel(T* __restrict__ out, const T* __restrict__ q_base, int 
   const int p = positions[tkn];
   const int slot = seq_slot[token_item[tkn]];
   const int* bt = block_table + (size_t)slot * bt_stride;
-  const int lo = window > 0 ? max(0, p - window + 1) : 0;
+  const int lo = mi::first_visible(p, window);
 
   const T* q = q_base + (size_t)tkn * q_stride + (size_t)head * hd;
   for (int d = lane; d < hd; d += 32) qs[warp][d] = mi::to_float(q[d]);
@@ -93,13 +98,14 @@ attention_generic_kernel(T* __restrict__ out, const T* __restrict__ q_base, int 
   const size_t head_off = (size_t)kvh * page_size * hd;
   const size_t v_off = (size_t)nkv * page_size * hd;
 
-  float o[MAX_HD / 32];
+  float o[HD_MAX / 32];
 #pragma unroll
-  for (int i = 0; i < MAX_HD / 32; ++i) o[i] = 0.f;
+  for (int i = 0; i < HD_MAX / 32; ++i) o[i] = 0.f;
   float m = -INFINITY, l = 0.f;
   if (sink) { m = sink[head]; l = 1.f; }
   const bool unnormalised = score_bias != nullptr;
   const float sb = unnormalised ? score_bias[head] : 0.f;
+  const float r1 = distance ? distance[head] : 0.f, r2 = distance ? distance[nh + head] : 0.f;
   if (unnormalised) m = 0.f;
 
   // two stretches of keys: the request's first keep_first keys that the window has passed (none without a window),
@@ -116,6 +122,7 @@ attention_generic_kernel(T* __restrict__ out, const T* __restrict__ q_base, int 
       koff = (long long)((size_t)page * page_elems + head_off + (size_t)(j % page_size) * hd);
       s = scale * dot_row<T>(kv_layer + koff, qs[warp], hd);
       if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+      if (distance) s -= r1 * log1pf(r2 * (float)(p - j));
     }
     float pe;
     if (unnormalised) {
@@ -127,7 +134,7 @@ attention_generic_kernel(T* __restrict__ out, const T* __restrict__ q_base, int 
       l = l * alpha + mi::warp_sum(pe);
       m = m_new;
 #pragma unroll
-      for (int i = 0; i < MAX_HD / 32; ++i) o[i] *= alpha;
+      for (int i = 0; i < HD_MAX / 32; ++i) o[i] *= alpha;
     }
     for (int jj = 0; jj < 32; ++jj) {
       const float pj = __shfl_sync(0xffffffffu, pe, jj);
@@ -135,7 +142,7 @@ attention_generic_kernel(T* __restrict__ out, const T* __restrict__ q_base, int 
       if (off < 0) continue;  // uniform over the warp
       const T* v = kv_layer + off + v_off;
 #pragma unroll
-      for (int i = 0; i < MAX_HD / 32; ++i) {
+      for (int i = 0; i < HD_MAX / 32; ++i) {
         const int d = lane + 32 * i;
         if (d < hd) o[i] = fmaf(pj, mi::to_float(v[d]), o[i]);
       }
@@ -143,13 +150,13 @@ attention_generic_kernel(T* __restrict__ out, const T* __restrict__ q_base, int 
   }
   const float inv = unnormalised ? 1.f : 1.f / l;
   T* dst = out + ((size_t)tkn * nh + head) * out_hd;
-  const T* gt = gate ? gate + (size_t)tkn * gate_stride + (size_t)head * out_hd : nullptr;
+  const T* gt = gate ? gate + (size_t)tkn * gate_stride : nullptr;
 #pragma unroll
-  for (int i = 0; i < MAX_HD / 32; ++i) {
+  for (int i = 0; i < HD_MAX / 32; ++i) {
     const int d = lane + 32 * i;
     if (d < out_hd) {
       float y = o[i] * inv;
-      if (gt) y = y / (1.f + expf(-mi::to_float(gt[d])));
+      if (gt) y = y / (1.f + expf(-mi::to_float(gt[mi::gate_index(head, d, out_hd, gate_per_head)])));
       dst[d] = mi::from_float<T>(y);
     }
   }
@@ -162,8 +169,10 @@ MI_API int mi_attention_generic(void* out, const void* q_base, int q_stride, int
                                 const int* block_table, int bt_stride, const int* token_item,
                                 const int* positions, const int* seq_slot, int T, int nh, int nkv, int hd,
                                 int page_size, float scale, int window, const float* sink, const void* gate,
-                                int gate_stride, int out_hd, int keep_first, float softcap, const float* score_bias, cudaStream_t stream) {
+                                int gate_stride, int out_hd, int keep_first, float softcap, const float* score_bias,
+                                int gate_per_head, const float* distance, cudaStream_t stream) {
   MI_REQUIRE(!(softcap < 0.f) && !(sink && score_bias), "attention: softcap=%f must not be negative, and unnormalised weights take no sink", softcap);
+  MI_REQUIRE(!(distance && score_bias), "attention: a distance bias goes with a softmax");
   MI_REQUIRE(keep_first >= 0, "attention: keep_first=%d must not be negative", keep_first);
   MI_REQUIRE(out_hd > 0 && out_hd <= hd, "attention: out_hd=%d must lie in 1..head_dim", out_hd);
   MI_REQUIRE(T >= 0 && nh > 0 && nkv > 0 && nh % nkv == 0, "attention: bad head counts nh=%d nkv=%d", nh, nkv);
@@ -172,17 +181,17 @@ MI_API int mi_attention_generic(void* out, const void* q_base, int q_stride, int
   MI_REQUIRE(T <= 65535, "attention: more than 65535 tokens in one launch (T=%d)", T);
   if (T == 0) return 0;
   dim3 grid((nh + WARPS - 1) / WARPS, T);
-  if (dtype == MI_BF16)
-    mi::launch(attention_generic_kernel<__nv_bfloat16>, dim3(grid), dim3(WARPS * 32), 0, stream, 
-        (__nv_bfloat16*)out, (const __nv_bfloat16*)q_base, q_stride, (const __nv_bfloat16*)kv_layer, block_table,
-        bt_stride, token_item, positions, seq_slot, nh, nkv, hd, page_size, scale, window, sink, (const __nv_bfloat16*)gate,
-        gate_stride, out_hd, keep_first, softcap, score_bias);
-  else if (dtype == MI_F32)
-    mi::launch(attention_generic_kernel<float>, dim3(grid), dim3(WARPS * 32), 0, stream, 
-        (float*)out, (const float*)q_base, q_stride, (const float*)kv_layer, block_table, bt_stride, token_item,
-        positions, seq_slot, nh, nkv, hd, page_size, scale, window, sink, (const float*)gate, gate_stride, out_hd, keep_first, softcap, score_bias);
+#define MI_GENERIC(TT, MAXHD)                                                                                              \
+  mi::launch(attention_generic_kernel<TT, MAXHD>, dim3(grid), dim3(WARPS * 32), 0, stream, (TT*)out, (const TT*)q_base, q_stride, \
+             (const TT*)kv_layer, block_table, bt_stride, token_item, positions, seq_slot, nh, nkv, hd, page_size, scale, window, \
+             sink, (const TT*)gate, gate_stride, out_hd, keep_first, softcap, score_bias, gate_per_head, distance)
+  if (dtype == MI_BF16 && hd <= 256) MI_GENERIC(__nv_bfloat16, 256);
+  else if (dtype == MI_BF16) MI_GENERIC(__nv_bfloat16, MAX_HD);
+  else if (dtype == MI_F32 && hd <= 256) MI_GENERIC(float, 256);
+  else if (dtype == MI_F32) MI_GENERIC(float, MAX_HD);
   else
     return mi_fail("attention: unknown dtype %d", dtype);
+#undef MI_GENERIC
   MI_LAUNCH_OK("attention_generic");
   return 0;
 }

@@ -19,10 +19,11 @@
 //
 // Options (off when null): a sink per query head joins the softmax's denominator once, at the end
 // (exp(sink), unscaled, no value); an output gate multiplies the output row with sigmoid(gate[token,
-// head, :]); out_hd < head size writes only the first out_hd values of a head (padded cache rows).
+// head, :]), or with one gate per head; out_hd < head size writes only the first out_hd values of a head (padded cache rows).
 //
 // Shaped scores (attention_scores.cuh): a cap on the scaled scores, and sigmoid weights that are not normalised over the
-// keys - the score enters the online softmax as the logarithm of its weight and the output is multiplied with 2^m at the end.
+// keys - the score enters the online softmax as the logarithm of its weight and the output is multiplied with 2^m at the end;
+// or a distance bias, which is taken off the scores of a softmax.
 //
 // Compiled once per head size: -DMI_HEAD_DIM=<multiple of 16, 16..256>.
 #include "attention_scores.cuh"
@@ -94,6 +95,8 @@ struct PrefillArgs {
   int gate_stride, out_hd;
   float scale, softcap;          // shaped scores: the scale itself and the cap (0: none)
   const float* score_bias;       // [nh]: sigmoid weights; null: softmax
+  int gate_per_head;             // one gate per head, head h at h
+  const float* distance;         // [2, nh] r1, r2 of the distance bias; or null
 };
 
 // Gathers keys kb*BK .. kb*BK+BK of one kv head (K and V) into a stage; rows past `last_key` are zeros.
@@ -133,7 +136,7 @@ attention_prefill_kernel(PrefillArgs a) {
   const int row0 = a.q_start[item] + off;
   const int p0 = a.ctx_len[item] - n_new + off;           // position of the tile's first row
   const int p_last = p0 + rows - 1;
-  const int lo_tile = a.window > 0 ? max(0, p0 - a.window + 1) : 0;
+  const int lo_tile = mi::first_visible(p0, a.window);
   const int kb_begin = lo_tile / BK, kb_end = p_last / BK;   // inclusive
   // key blocks of the request's first keep_first keys that lie before the window's first block come first
   const int n_first = (a.window > 0 && a.keep_first > 0) ? min((a.keep_first - 1) / BK + 1, kb_begin) : 0;
@@ -164,6 +167,9 @@ attention_prefill_kernel(PrefillArgs a) {
   const bool row_ok[2] = {warp * 16 + g < rows, warp * 16 + g + 8 < rows};
   const bool shaped = SHAPED, sigmoid = SHAPED && a.score_bias != nullptr;
   const float head_bias = sigmoid ? a.score_bias[head] : 0.f;
+  const bool distance = SHAPED && a.distance != nullptr;
+  const float r1 = distance ? a.distance[head] : 0.f, r2 = distance ? a.distance[a.nh + head] : 0.f;
+  const int lo_row[2] = {mi::first_visible(pr[0], a.window), mi::first_visible(pr[1], a.window)};
 
   // ldmatrix lane addressing: lane l gives the row address of 8x8 matrix l/8, row l%8
   const int lm = lane >> 3, lr = lane & 7;
@@ -221,8 +227,9 @@ attention_prefill_kernel(PrefillArgs a) {
       for (int c = 0; c < 4; ++c) {
         const int j = kb * BK + i * 8 + 2 * t + (c & 1);
         const int h = c >> 1;
-        const bool see = row_ok[h] && j <= pr[h] && (a.window <= 0 || j > pr[h] - a.window || j < a.keep_first);
-        const float v = see ? (shaped ? mi::shaped_logit2(s[i][c], a.scale, a.softcap, sigmoid, head_bias) : s[i][c] * a.scale_log2) : -INFINITY;
+        const bool see = row_ok[h] && j <= pr[h] && (j >= lo_row[h] || (a.window > 0 && j < a.keep_first));
+        float v = see ? (shaped ? mi::shaped_logit2(s[i][c], a.scale, a.softcap, sigmoid, head_bias) : s[i][c] * a.scale_log2) : -INFINITY;
+        if (distance && see) v -= mi::distance_logit2(r1, r2, pr[h] - j);
         s[i][c] = v;
         mx[h] = fmaxf(mx[h], v);
       }
@@ -291,15 +298,16 @@ attention_prefill_kernel(PrefillArgs a) {
     // sigmoid weights: the sums hold weight * 2^(-m); nothing is divided by the weights' sum
     const float inv = sigmoid ? (m_run[h] == -INFINITY ? 0.f : exp2f(m_run[h])) : f / l;
     const size_t r = (size_t)(row0 + warp * 16 + g + 8 * h);
+    const float head_gate = a.gate && a.gate_per_head ? __bfloat162float(a.gate[r * a.gate_stride + head]) : 0.f;
     __nv_bfloat16* dst = a.out + (r * a.nh + head) * a.out_hd;
-    const __nv_bfloat16* gt = a.gate ? a.gate + r * a.gate_stride + (size_t)head * a.out_hd : nullptr;
+    const __nv_bfloat16* gt = a.gate ? a.gate + r * a.gate_stride + (size_t)head * a.out_hd : nullptr;      // (a gate per value)
 #pragma unroll
     for (int i = 0; i < NT_O; ++i) {
       const int d = i * 8 + 2 * t;
       if (d >= a.out_hd) continue;
       float y0 = o[i][2 * h] * inv, y1 = o[i][2 * h + 1] * inv;
       if (gt) {
-        const float2 gg = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gt + d));
+        const float2 gg = a.gate_per_head ? make_float2(head_gate, head_gate) : __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gt + d));
         y0 = __fdividef(y0, 1.f + __expf(-gg.x));
         y1 = __fdividef(y1, 1.f + __expf(-gg.y));
       }
@@ -317,10 +325,11 @@ MI_API int mi_attention_prefill_bf16(void* out, const void* q_base, int q_stride
                                      const int* q_start, const int* q_len, const int* ctx_len, const int* seq_slot,
                                      int nh, int nkv, int page_size, float scale, int window, const float* sink,
                                      const void* gate, int gate_stride, int out_hd, int keep_first, float softcap,
-                                     const float* score_bias, cudaStream_t stream) {
+                                     const float* score_bias, int gate_per_head, const float* distance, cudaStream_t stream) {
   MI_REQUIRE(!(softcap < 0.f) && !(sink && score_bias), "attention_prefill: softcap must not be negative, and sigmoid weights take no sink");
+  MI_REQUIRE(!(distance && score_bias), "attention_prefill: a distance bias goes with a softmax");
   MI_REQUIRE(keep_first >= 0, "attention_prefill: keep_first=%d must not be negative", keep_first);
-  MI_REQUIRE(out_hd > 0 && out_hd <= HD && out_hd % 2 == 0 && gate_stride % 2 == 0, "attention_prefill: out_hd=%d must be even, up to %d", out_hd, HD);
+  MI_REQUIRE(out_hd > 0 && out_hd <= HD && out_hd % 2 == 0 && (gate_per_head || gate_stride % 2 == 0), "attention_prefill: out_hd=%d must be even, up to %d", out_hd, HD);
   MI_REQUIRE(n_tiles >= 0 && nh > 0 && nkv > 0 && nh % nkv == 0, "attention_prefill: bad head counts nh=%d nkv=%d", nh, nkv);
   MI_REQUIRE(page_size > 0 && q_stride % 8 == 0, "attention_prefill: bad page_size=%d or q_stride=%d", page_size, q_stride);
   MI_REQUIRE(nh <= 65535, "attention_prefill: too many heads for one launch");
@@ -337,7 +346,7 @@ MI_API int mi_attention_prefill_bf16(void* out, const void* q_base, int q_stride
   a.nh = nh; a.nkv = nkv; a.page_size = page_size; a.window = window; a.keep_first = keep_first;
   a.scale_log2 = scale * 1.4426950408889634f;
   a.sink = sink; a.gate = (const __nv_bfloat16*)gate; a.gate_stride = gate_stride; a.out_hd = out_hd;
-  a.scale = scale; a.softcap = softcap; a.score_bias = score_bias;
+  a.scale = scale; a.softcap = softcap; a.score_bias = score_bias; a.gate_per_head = gate_per_head; a.distance = distance;
   const size_t smem = (size_t)(BQ + 4 * BK) * LDS * sizeof(__nv_bfloat16);
   static bool configured = false;
   if (!configured) {
@@ -346,7 +355,7 @@ MI_API int mi_attention_prefill_bf16(void* out, const void* q_base, int q_stride
     if (e != cudaSuccess) return mi_fail("attention_prefill: cannot get %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
     configured = true;
   }
-  if (softcap > 0.f || score_bias != nullptr) mi::launch(attention_prefill_kernel<true>, dim3(dim3(n_tiles, nh)), dim3(WARPS * 32), smem, stream, a);
+  if (softcap > 0.f || score_bias != nullptr || distance != nullptr) mi::launch(attention_prefill_kernel<true>, dim3(dim3(n_tiles, nh)), dim3(WARPS * 32), smem, stream, a);
   else mi::launch(attention_prefill_kernel<false>, dim3(dim3(n_tiles, nh)), dim3(WARPS * 32), smem, stream, a);
   MI_LAUNCH_OK("attention_prefill");
   return 0;

@@ -177,6 +177,8 @@ struct Args {
   // output to rescale - and the output rows are stored as the products leave them.
   float scale, softcap;
   const float* score_bias;
+  int gate_per_head;             // one gate per head, head h at h, instead of one per value
+  const float* distance;         // [2, nh] r1, r2 of a distance bias taken off the scores of a softmax; or null
 };
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -426,8 +428,8 @@ __device__ __forceinline__ Work work_of(const Args& a, int w, int rank) {
   k.rows_tok = min(tok_per_block, qlen - k.o);            // tokens of this work that exist
   k.p_first = k.start + k.o;
   k.p_last = k.start + k.o + k.rows_tok - 1;
-  const int lo_first = a.window > 0 ? max(0, k.p_first - a.window + 1) : 0;
-  k.lo_last = a.window > 0 ? max(0, k.p_last - a.window + 1) : 0;
+  const int lo_first = mi::first_visible(k.p_first, a.window);
+  k.lo_last = mi::first_visible(k.p_last, a.window);
   k.t_begin = lo_first / BN;
   k.n_first = (a.window > 0 && a.keep_first > 0) ? min((a.keep_first - 1) / BN + 1, k.t_begin) : 0;
   k.n = k.n_first + k.p_last / BN - k.t_begin + 1;        // key tiles to walk: the i-th is tile i < n_first ? i : t_begin + i - n_first
@@ -444,7 +446,8 @@ __device__ __forceinline__ int nth_work(int i, int b, int blocks, int total) {
   return w < total ? w : -1;
 }
 
-// SCORES: 0 - the softmax of the scaled scores; 1 - of capped scores; 2 - sigmoid weights (capped or not).  The forms for
+// SCORES: 0 - the softmax of the scaled scores; 1 - of capped scores; 2 - sigmoid weights (capped or not); 3 - the softmax of
+// (capped or uncapped) scores less a distance bias.  The forms for
 // shaped scores are compiled apart: as branches on values of Args in the one kernel they cost the plain softmax a quarter of
 // its speed.
 template <int CTAS, int SCORES = 0>
@@ -662,7 +665,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
     const int q = warp & 3, st = warp >> 2;
     const int r = q * 32 + lane;                           // row of the block = lane of the tensor memory
     const uint32_t t_lane = tmem_base + ((uint32_t)(q * 32) << 16);
-    constexpr bool shaped = SCORES != 0, sigmoid = SCORES == 2;
+    constexpr bool shaped = SCORES != 0, sigmoid = SCORES == 2, distance = SCORES == 3;
     const float sc = shaped ? 1.f : a.scale_log2;          // shaped scores come as base-2 logits already
     int o_seen = 0;
     auto wait_o = [&](int upto) {
@@ -688,10 +691,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
       const int head = wk.head0 + (a.hpt == 2 ? (r >> 6) : 0);
       const bool row_valid = tok < rows_tok;
       const int pos = row_valid ? start + o + tok : p_last;
-      const int lo_r = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+      const int lo_r = mi::first_visible(pos, a.window);
       float m_run = -INFINITY, l_run = 0.f;
       const int n_mine = (n - st + 1) / 2;                 // tiles of this stream
       const float head_bias = sigmoid ? a.score_bias[head] : 0.f;
+      const float r1 = distance ? a.distance[head] : 0.f, r2 = distance ? a.distance[a.nh + head] : 0.f;
 
       for (int k = 0; k < n_mine; ++k) {
         const int j = 2 * k + st;
@@ -709,6 +713,17 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
         if (sigmoid) {
 #pragma unroll
           for (int e = 0; e < BN; ++e) v[e] = mi::shaped_sigmoid_weight(v[e], a.scale, a.softcap, head_bias);
+        } else if (distance) {
+          // keys behind the query only: what lies ahead (a logarithm of nothing) is hidden below
+          const float at0 = fmaf(r2, (float)(pos - key0), 1.f);      // 1 + r2 d of the tile's first key
+          if (a.softcap > 0.f) {
+#pragma unroll
+            for (int e = 0; e < BN; ++e)
+              v[e] = fmaf(-r1, mi::lg2_fast(fmaf(-r2, (float)e, at0)), mi::shaped_logit2(v[e], a.scale, a.softcap, false, 0.f));
+          } else {
+#pragma unroll
+            for (int e = 0; e < BN; ++e) v[e] = fmaf(-r1, mi::lg2_fast(fmaf(-r2, (float)e, at0)), v[e] * a.scale_log2);
+          }
         } else if (shaped) {
 #pragma unroll
           for (int e = 0; e < BN; ++e) v[e] = mi::shaped_logit2(v[e], a.scale, a.softcap, false, 0.f);
@@ -844,7 +859,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
           const int head2 = wk.head0 + (a.hpt == 2 ? (rg >> 6) : 0);
           if (tok2 < rows_tok) {
             uint4 wv = *reinterpret_cast<const uint4*>(mine + rw * OUT_ROW_BYTES + ((chunk ^ (rw & (CH - 1))) << 4));
-            if (a.gate) {
+            if (a.gate && a.gate_per_head) {
+              const __nv_bfloat16 hg = a.gate[(size_t)(wk.row0 + tok2) * a.gate_stride + head2];
+              const __nv_bfloat162 hg2 = __halves2bfloat162(hg, hg);
+              const uint32_t gw = *reinterpret_cast<const uint32_t*>(&hg2);
+              wv.x = gate_pair(wv.x, gw); wv.y = gate_pair(wv.y, gw); wv.z = gate_pair(wv.z, gw); wv.w = gate_pair(wv.w, gw);
+            } else if (a.gate) {
               const uint4 gv = *reinterpret_cast<const uint4*>(a.gate + (size_t)(wk.row0 + tok2) * a.gate_stride + (size_t)head2 * HD + st * OD + chunk * 8);
               wv.x = gate_pair(wv.x, gv.x); wv.y = gate_pair(wv.y, gv.y); wv.z = gate_pair(wv.z, gv.z); wv.w = gate_pair(wv.w, gv.w);
             }
@@ -973,11 +993,12 @@ MI_API int mi_attention_prefill_tc(void* out, const void* q_map, const void* kv_
                                    const int* seq_slot, int* status, int nh, int nkv, int page_size, float scale, int window,
                                    int num_sms, cudaStream_t stream, const int* tiles128, int n_tiles128, int pairs,
                                    const float* sink, const void* gate, int gate_stride, int keep_first, float softcap,
-                                   const float* score_bias) {
+                                   const float* score_bias, int gate_per_head, const float* distance) {
   MI_REQUIRE(!(softcap < 0.f) && !(sink && score_bias), "attention_prefill_tc: softcap must not be negative, and sigmoid weights take no sink");
+  MI_REQUIRE(!(distance && score_bias), "attention_prefill_tc: a distance bias goes with a softmax");
   MI_REQUIRE(keep_first >= 0, "attention_prefill_tc: keep_first=%d must not be negative", keep_first);
   MI_REQUIRE(num_sms > 0, "attention_prefill_tc: num_sms");
-  MI_REQUIRE(gate == nullptr || (((uintptr_t)gate % 16) == 0 && gate_stride % 8 == 0), "attention_prefill_tc: the gate rows must be 16-byte aligned");
+  MI_REQUIRE(gate == nullptr || gate_per_head || (((uintptr_t)gate % 16) == 0 && gate_stride % 8 == 0), "attention_prefill_tc: the gate rows must be 16-byte aligned");
   MI_REQUIRE(n_tiles >= 0 && nh > 0 && nkv > 0 && nh % nkv == 0, "attention_prefill_tc: bad head counts nh=%d nkv=%d", nh, nkv);
   MI_REQUIRE(page_size % 64 == 0, "attention_prefill_tc: page_size=%d must be a multiple of 64", page_size);
   MI_REQUIRE(scale > 0.f, "attention_prefill_tc: the scale must be positive");
@@ -996,12 +1017,12 @@ MI_API int mi_attention_prefill_tc(void* out, const void* q_map, const void* kv_
   a.n_tiles = n_tiles; a.nh = nh; a.nkv = nkv; a.page_size = page_size; a.window = window; a.keep_first = keep_first;
   a.scale_log2 = scale * 1.4426950408889634f;
   a.sink = sink; a.gate = (const __nv_bfloat16*)gate; a.gate_stride = gate_stride;
-  a.scale = scale; a.softcap = softcap; a.score_bias = score_bias;
+  a.scale = scale; a.softcap = softcap; a.score_bias = score_bias; a.gate_per_head = gate_per_head; a.distance = distance;
   CUtensorMap qm, km;
   memcpy(&qm, q_map, sizeof(qm));
   memcpy(&km, kv_map, sizeof(km));
   const bool even_group = (nh / nkv) % 2 == 0;
-  const int scores = score_bias != nullptr ? 2 : (softcap > 0.f ? 1 : 0);
+  const int scores = score_bias != nullptr ? 2 : (distance != nullptr ? 3 : (softcap > 0.f ? 1 : 0));
   bool placed = false;
   if (pairs && HD == 128 && even_group && num_sms >= 2 && tiles128 != nullptr && n_tiles128 > 0) {
     // a pair of blocks: 128 tokens of two neighbouring heads, a head each
@@ -1011,7 +1032,8 @@ MI_API int mi_attention_prefill_tc(void* out, const void* q_map, const void* kv_
     p.hpt = 1;
     p.hw = 2;
     p.skip_odd = 0;
-    const int r = scores == 2 ? launch_prefill_tc<2, 2>(qm, km, p, num_sms, stream, &placed)
+    const int r = scores == 3 ? launch_prefill_tc<2, 3>(qm, km, p, num_sms, stream, &placed)
+                : scores == 2 ? launch_prefill_tc<2, 2>(qm, km, p, num_sms, stream, &placed)
                 : scores == 1 ? launch_prefill_tc<2, 1>(qm, km, p, num_sms, stream, &placed) : launch_prefill_tc<2>(qm, km, p, num_sms, stream, &placed);
     if (r != 0) return r;
   }
@@ -1024,7 +1046,8 @@ MI_API int mi_attention_prefill_tc(void* out, const void* q_map, const void* kv_
       a.n_tiles = n_tiles128;
       a.skip_odd = 0;
     }
-    const int r = scores == 2 ? launch_prefill_tc<1, 2>(qm, km, a, num_sms, stream, &placed)
+    const int r = scores == 3 ? launch_prefill_tc<1, 3>(qm, km, a, num_sms, stream, &placed)
+                : scores == 2 ? launch_prefill_tc<1, 2>(qm, km, a, num_sms, stream, &placed)
                 : scores == 1 ? launch_prefill_tc<1, 1>(qm, km, a, num_sms, stream, &placed) : launch_prefill_tc<1>(qm, km, a, num_sms, stream, &placed);
     if (r != 0) return r;
   }

@@ -556,16 +556,17 @@ MI_API int mi_gemm_tc_glu_bf16(void* out, const void* x, const void* w, int M, i
 // The grouped form: x [M, K] holds rows sorted by expert, every expert's rows starting at a multiple of tile_rows (a
 // multiple of 256); tile_expert [M / tile_rows] (device) names the expert of each stretch, -1 where nobody owns the rows;
 // w stacks the experts' matrices ([experts, 2 N, K] with SwiGLU, gate rows then up rows; [experts, N, K] without).
-// glu, limit: the gated activation of the SwiGLU form (a MiGlu of common.cuh).
+// glu, limit: the gated activation of the SwiGLU form (a MiGlu of common.cuh).  relu2: without SwiGLU, max(bf16(x w^T), 0)^2 is
+// written instead of the product.
 MI_API int mi_gemm_tc_grouped_bf16(void* out, const void* x, const void* w, int M, int N, int K, int ldo, int experts, int swiglu,
-                                   const int* tile_expert, int tile_rows, int* status, int pairs, int glu, float limit, cudaStream_t stream) {
+                                   const int* tile_expert, int tile_rows, int* status, int pairs, int glu, float limit, int relu2, cudaStream_t stream) {
   MI_REQUIRE(glu == MI_GLU_SILU || (glu == MI_GLU_CLAMPED && limit > 0.f), "gemm_tc_grouped: unknown activation %d or a limit that is not positive", glu);
   MI_REQUIRE(experts > 0 && tile_expert != nullptr && tile_rows > 0 && tile_rows % 256 == 0 && M % tile_rows == 0,
              "gemm_tc_grouped: rows=%d must come in stretches of tile_rows=%d, a multiple of 256", M, tile_rows);
   if (swiglu && glu == MI_GLU_CLAMPED)
     return run<true, true, MI_GLU_CLAMPED>(out, x, w, M, N, K, ldo, status, pairs, stream, experts, tile_expert, tile_rows, 0, glu, limit);
   return swiglu ? run<true, true>(out, x, w, M, N, K, ldo, status, pairs, stream, experts, tile_expert, tile_rows)
-                : run<false, true>(out, x, w, M, N, K, ldo, status, pairs, stream, experts, tile_expert, tile_rows);
+                : run<false, true>(out, x, w, M, N, K, ldo, status, pairs, stream, experts, tile_expert, tile_rows, relu2 ? 1 : 0);
 }
 
 // out[M, N] = x w^T, all bf16.

@@ -5,12 +5,13 @@
 //            multiply exactly in float32, so this is the 32-bit sum of the rounded inputs.)  One warp per token: scores
 //            s = sigmoid(z), choice = s + correction; the `top` experts of largest choice (ties: the lower
 //            index); weights = their s divided by (the sum of those s + 1e-20).  Or (mode 1) the `top` largest logits
-//            are chosen and the weights are the softmax over the chosen logits alone.
+//            are chosen and the weights are the softmax over the chosen logits alone.  A constant may multiply the weights.
 //   align    one block: counts the (token, choice) pairs of every expert, gives each expert a range of
 //            rows rounded up to the row tile, and every pair a row in its expert's range.  Rows nobody
 //            owns are marked -1, tiles nobody owns too; the grid of the products is sized for the worst case.
 //   gate-up  grouped product: a block takes one row tile (rows of ONE expert, gathered from the tokens'
-//            normalised rows) and a slice of that expert's gate and up rows, and writes silu(g) * u.
+//            normalised rows) and a slice of that expert's gate and up rows, and writes silu(g) * u.  Experts without a
+//            gate have an up matrix alone, and what is written is its product's activation (squared ReLU).
 //   down     grouped product of those rows with the expert's down matrix, written as float32.
 //   combine  out[token] = sum over its choices, in the order of the choices, of weight * down row.
 //
@@ -28,7 +29,7 @@ constexpr int ROUTE_WARPS = 8;
 // A warp per token: a lane keeps the scores of the experts lane, lane + 32, ... (up to eight) and the warp picks the
 // `top` largest choices one after the other.
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
-moe_route_kernel(const float* __restrict__ z, int z_stride, int Tn, const float* __restrict__ corr, int E, int top, int mode,
+moe_route_kernel(const float* __restrict__ z, int z_stride, int Tn, const float* __restrict__ corr, int E, int top, int mode, float mult,
                  int* __restrict__ idx_out, float* __restrict__ w_out) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int t = blockIdx.x * ROUTE_WARPS + warp;
@@ -72,7 +73,7 @@ moe_route_kernel(const float* __restrict__ z, int z_stride, int Tn, const float*
     for (int i = 0; i < MAX_EXPERTS / 32; ++i)
       if (lane + 32 * i == bi) choice[i] = -INFINITY;
   }
-  if (lane < top) w_out[(size_t)t * top + lane] = mode == 1 ? mine / sum : mine / (sum + 1e-20f);
+  if (lane < top) w_out[(size_t)t * top + lane] = mult * (mode == 1 ? mine / sum : mine / (sum + 1e-20f));
 }
 
 __global__ void __launch_bounds__(1024)
@@ -178,14 +179,22 @@ constexpr int GBK = 64;          // k per stage
 constexpr int GLDS = GBK + 8;    // shared-memory row stride in elements (odd number of 16-byte units)
 constexpr int WN_COLS = 32;      // columns of a warp's tile
 
-// WM x WN warps; a warp owns 16 rows x 32 columns (of gate and of up, if SWIGLU).  Block tile: 16 WM rows x 32 WN columns.
+// What a grouped product leaves: float32 rows (the down product), the gated activation of a gate and an up product, or the
+// activation of an up product alone (squared ReLU).
+enum GroupedMode { PLAIN = 0, GATED = 1, ACTIVATED = 2 };
+__device__ __forceinline__ float relu_squared(float x) {
+  x = fmaxf(x, 0.f);
+  return x * x;
+}
+
+// WM x WN warps; a warp owns 16 rows x 32 columns (of gate and of up, if GATED).  Block tile: 16 WM rows x 32 WN columns.
 // STAGES slices of 64 elements of K are in flight: with few rows an expert the kernel streams weights, and what a block
 // has asked for is what keeps the memory busy - narrow tiles take more stages.
-template <int WM, int WN, bool SWIGLU, int STAGES>
+template <int WM, int WN, int MODE, int STAGES>
 __global__ void __launch_bounds__(WM * WN * 32)
 moe_gemm_bf16_kernel(GroupedArgs a) {
   constexpr int TM = 16 * WM, BN = WN_COLS * WN, THREADS = WM * WN * 32;
-  constexpr int NB = SWIGLU ? 2 : 1;
+  constexpr int NB = MODE == GATED ? 2 : 1;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   __nv_bfloat16* as = reinterpret_cast<__nv_bfloat16*>(smem_raw);        // [STAGES][TM][GLDS]
   __nv_bfloat16* bs = as + STAGES * TM * GLDS;                           // [STAGES][NB][BN][GLDS]
@@ -279,9 +288,9 @@ moe_gemm_bf16_kernel(GroupedArgs a) {
     for (int i = 0; i < 4; ++i) {
       const int n = n0 + wn * WN_COLS + i * 8 + 2 * t;
       if (n >= N) continue;
-      if (SWIGLU) {
-        const float y0 = mi::glu_fast(acc[0][i][2 * h], acc[1][i][2 * h], a.glu, a.limit);
-        const float y1 = mi::glu_fast(acc[0][i][2 * h + 1], acc[1][i][2 * h + 1], a.glu, a.limit);
+      if (MODE != PLAIN) {
+        const float y0 = MODE == ACTIVATED ? relu_squared(acc[0][i][2 * h]) : mi::glu_fast(acc[0][i][2 * h], acc[NB - 1][i][2 * h], a.glu, a.limit);
+        const float y1 = MODE == ACTIVATED ? relu_squared(acc[0][i][2 * h + 1]) : mi::glu_fast(acc[0][i][2 * h + 1], acc[NB - 1][i][2 * h + 1], a.glu, a.limit);
         __nv_bfloat16* o = (__nv_bfloat16*)a.out + orow + n;
         o[0] = __float2bfloat16_rn(y0);
         if (n + 1 < N) o[1] = __float2bfloat16_rn(y1);
@@ -298,7 +307,7 @@ moe_gemm_bf16_kernel(GroupedArgs a) {
 // global memory straight to the registers of the warp that multiplies them - 16-byte loads that bypass L1, four slices
 // of K asked for before the first is used - as in the engine's few-row product for dense matrices.  A block of eight
 // warps owns a row tile of 16 rows and 8 * (8 / KS) output columns; KS warps share a group of 8 columns (of gate and
-// of up, if SWIGLU) and deal the 32-element slices of K among them, and their partial tiles are added through shared
+// of up, if GATED) and deal the 32-element slices of K among them, and their partial tiles are added through shared
 // memory in the order of the warps, so a value is a function of (N, K) alone.  The k index inside a slice is permuted
 // the same way for both operands, so that a thread's 16-byte load is its fragment of two consecutive MMAs.
 __device__ __forceinline__ uint4 ld_stream16(const void* p) {
@@ -309,10 +318,10 @@ __device__ __forceinline__ uint4 ld_stream16(const void* p) {
 
 constexpr int SW = 8;       // warps of a block of the streaming product
 
-template <bool SWIGLU, int KS>
+template <int MODE, int KS>
 __global__ void __launch_bounds__(SW * 32)
 moe_stream_bf16_kernel(GroupedArgs a) {
-  constexpr int NB = SWIGLU ? 2 : 1, GROUPS = SW / KS, U = 4;
+  constexpr int NB = MODE == GATED ? 2 : 1, GROUPS = SW / KS, U = 4;
   __shared__ float red[SW][16][NB * 8 + 1];
   __shared__ int s_row[16];
   const int tile = blockIdx.y;
@@ -391,7 +400,8 @@ moe_stream_bf16_kernel(GroupedArgs a) {
       for (int k = 0; k < KS; ++k) v[b] += red[grp * KS + k][r][b * 8 + c];
     }
     const size_t o = (size_t)(tile * 16 + r) * N + n;
-    if (SWIGLU) ((__nv_bfloat16*)a.out)[o] = __float2bfloat16_rn(mi::glu_fast(v[0], v[NB - 1], a.glu, a.limit));
+    if (MODE == GATED) ((__nv_bfloat16*)a.out)[o] = __float2bfloat16_rn(mi::glu_fast(v[0], v[NB - 1], a.glu, a.limit));
+    else if (MODE == ACTIVATED) ((__nv_bfloat16*)a.out)[o] = __float2bfloat16_rn(relu_squared(v[0]));
     else ((float*)a.out)[o] = v[0];
   }
 }
@@ -399,10 +409,10 @@ moe_stream_bf16_kernel(GroupedArgs a) {
 // float32: 16 rows x 64 columns per block of 256 threads, a thread one row x 4 columns; sums in the order of k
 constexpr int FTM = 16, FBN = 64, FBK = 16;
 
-template <bool SWIGLU>
+template <int MODE>
 __global__ void __launch_bounds__(256)
 moe_gemm_f32_kernel(GroupedArgs a) {
-  constexpr int NB = SWIGLU ? 2 : 1;
+  constexpr int NB = MODE == GATED ? 2 : 1;
   __shared__ float as[FTM][FBK + 1];
   __shared__ float bs[NB][FBN][FBK + 1];
   __shared__ int s_row[FTM];
@@ -452,7 +462,7 @@ moe_gemm_f32_kernel(GroupedArgs a) {
 #pragma unroll
   for (int c = 0; c < 4; ++c) {
     const int n = n0 + cg * 4 + c;
-    if (n < N) o[n] = SWIGLU ? mi::glu_exact(acc[0][c], acc[NB - 1][c], a.glu, a.limit) : acc[0][c];
+    if (n < N) o[n] = MODE == GATED ? mi::glu_exact(acc[0][c], acc[NB - 1][c], a.glu, a.limit) : (MODE == ACTIVATED ? relu_squared(acc[0][c]) : acc[0][c]);
   }
 }
 
@@ -486,17 +496,17 @@ moe_gather_kernel(__nv_bfloat16* __restrict__ xs, const __nv_bfloat16* __restric
   for (int i = threadIdx.x; i < H8; i += blockDim.x) dst[i] = src ? src[i] : make_uint4(0, 0, 0, 0);
 }
 
-template <int WM, int WN, bool SWIGLU, int STAGES>
+template <int WM, int WN, int MODE, int STAGES>
 int launch_bf16(const GroupedArgs& a, int tiles, cudaStream_t stream) {
   constexpr int TM = 16 * WM, BN = WN_COLS * WN;
-  const size_t smem = (size_t)STAGES * (TM + (SWIGLU ? 2 : 1) * BN) * GLDS * sizeof(__nv_bfloat16);
+  const size_t smem = (size_t)STAGES * (TM + (MODE == GATED ? 2 : 1) * BN) * GLDS * sizeof(__nv_bfloat16);
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(moe_gemm_bf16_kernel<WM, WN, SWIGLU, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(moe_gemm_bf16_kernel<WM, WN, MODE, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return mi_fail("moe_gemm: cannot get %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
     configured = true;
   }
-  mi::launch(moe_gemm_bf16_kernel<WM, WN, SWIGLU, STAGES>, dim3((a.N + BN - 1) / BN, tiles), dim3(WM * WN * 32), smem, stream, a);
+  mi::launch(moe_gemm_bf16_kernel<WM, WN, MODE, STAGES>, dim3((a.N + BN - 1) / BN, tiles), dim3(WM * WN * 32), smem, stream, a);
   return 0;
 }
 
@@ -510,14 +520,15 @@ MI_API int mi_moe_row_tile(int n_pairs, int E, int dtype) {
 
 // z: the router's logits in float32, rows of z_stride >= E values (a product of the engine's own: W_router h with float32
 // accumulation).  mode 0: sigmoid scores, chosen by score + correction, weights the scores over their sum; mode 1: the
-// largest logits are chosen (correction, if given, added for the choice), weights the softmax over the chosen logits.
-MI_API int mi_moe_route(const float* z, int z_stride, int T, const float* correction, int E, int top, int mode, int* idx_out, float* w_out,
+// largest logits are chosen (correction, if given, added for the choice), weights the softmax over the chosen logits.  The
+// weights are multiplied with mult.
+MI_API int mi_moe_route(const float* z, int z_stride, int T, const float* correction, int E, int top, int mode, float mult, int* idx_out, float* w_out,
                         cudaStream_t stream) {
   MI_REQUIRE((mode == 0 || mode == 1) && z_stride >= E, "moe_route: mode %d is not known or rows of %d logits are too short", mode, z_stride);
   MI_REQUIRE(T >= 0 && E > 0 && E <= MAX_EXPERTS, "moe_route: experts=%d must lie in 1..%d", E, MAX_EXPERTS);
   MI_REQUIRE(top > 0 && top <= E && top <= 32, "moe_route: top=%d must lie in 1..min(experts, 32)", top);
   if (T == 0) return 0;
-  mi::launch(moe_route_kernel, dim3((T + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), 0, stream, z, z_stride, T, correction, E, top, mode, idx_out, w_out);
+  mi::launch(moe_route_kernel, dim3((T + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), 0, stream, z, z_stride, T, correction, E, top, mode, mult, idx_out, w_out);
   MI_LAUNCH_OK("moe_route");
   return 0;
 }
@@ -535,29 +546,32 @@ MI_API int mi_moe_align(const int* topk_idx, int n_pairs, int E, int TM, int* so
   return 0;
 }
 
-// swiglu 1: out[row, :N] = act(a w_gate^T) * (a w_up^T), the expert's matrix holding N gate rows and then N up rows,
-// rows gathered from the tokens, the gated activation `glu` (a MiGlu) with its `limit`; swiglu 0: out[row, :N] = a w^T in
-// float32, rows by position.
+// mode 1: out[row, :N] = act(a w_gate^T) * (a w_up^T), the expert's matrix holding N gate rows and then N up rows,
+// rows gathered from the tokens, the gated activation `glu` (a MiGlu) with its `limit`; mode 2: out[row, :N] =
+// max(a w^T, 0)^2, the expert's matrix holding N rows, rows gathered; mode 0: out[row, :N] = a w^T in float32, rows by position.
 MI_API int mi_moe_gemm(const void* a_rows, int dtype, int a_stride, const void* w, void* out, const int* sorted_pair,
-                       const int* tile_expert, int max_tiles, int TM, int N, int K, int top, int swiglu, int glu, float limit,
+                       const int* tile_expert, int max_tiles, int TM, int N, int K, int top, int mode, int glu, float limit,
                        cudaStream_t stream) {
   MI_REQUIRE(glu == MI_GLU_SILU || (glu == MI_GLU_CLAMPED && limit > 0.f), "moe_gemm: unknown activation %d or a limit that is not positive", glu);
+  MI_REQUIRE(mode >= PLAIN && mode <= ACTIVATED, "moe_gemm: unknown mode %d", mode);
   MI_REQUIRE(N > 0 && K > 0 && max_tiles >= 0 && max_tiles <= 65535, "moe_gemm: bad sizes N=%d K=%d tiles=%d", N, K, max_tiles);
   if (max_tiles == 0) return 0;
   GroupedArgs g;
   g.a = a_rows; g.a_stride = a_stride; g.w = w; g.out = out; g.sorted_pair = sorted_pair; g.tile_expert = tile_expert;
-  g.N = N; g.K = K; g.top = top; g.gather = swiglu ? 1 : 0; g.glu = glu; g.limit = limit;
-  g.w_expert_stride = (long long)(swiglu ? 2 : 1) * N * K;
+  g.N = N; g.K = K; g.top = top; g.gather = mode != PLAIN ? 1 : 0; g.glu = glu; g.limit = limit;
+  g.w_expert_stride = (long long)(mode == GATED ? 2 : 1) * N * K;
   if (dtype == MI_F32) {
     MI_REQUIRE(TM == FTM, "moe_gemm: the float32 product takes row tiles of %d", FTM);
     const dim3 grid((N + FBN - 1) / FBN, max_tiles);
-    if (swiglu) mi::launch(moe_gemm_f32_kernel<true>, grid, dim3(256), 0, stream, g);
-    else mi::launch(moe_gemm_f32_kernel<false>, grid, dim3(256), 0, stream, g);
+    if (mode == GATED) mi::launch(moe_gemm_f32_kernel<GATED>, grid, dim3(256), 0, stream, g);
+    else if (mode == ACTIVATED) mi::launch(moe_gemm_f32_kernel<ACTIVATED>, grid, dim3(256), 0, stream, g);
+    else mi::launch(moe_gemm_f32_kernel<PLAIN>, grid, dim3(256), 0, stream, g);
   } else if (dtype == MI_BF16) {
     MI_REQUIRE(K % 8 == 0 && a_stride % 8 == 0, "moe_gemm: K=%d and the row stride %d must be multiples of 8 in bfloat16", K, a_stride);
     MI_REQUIRE(((uintptr_t)a_rows % 16) == 0 && ((uintptr_t)w % 16) == 0, "moe_gemm: operands must be 16-byte aligned");
     int rc;
-    if (TM == 64) rc = swiglu ? launch_bf16<4, 2, true, 3>(g, max_tiles, stream) : launch_bf16<4, 2, false, 3>(g, max_tiles, stream);
+    if (TM == 64) rc = mode == GATED ? launch_bf16<4, 2, GATED, 3>(g, max_tiles, stream)
+                  : mode == ACTIVATED ? launch_bf16<4, 2, ACTIVATED, 3>(g, max_tiles, stream) : launch_bf16<4, 2, PLAIN, 3>(g, max_tiles, stream);
     else if (TM == 16) {
       // few rows an expert: the weights are streamed once, straight into registers; K is dealt to eight warps where it
       // is long, to four (two groups of columns a block) where it is short
@@ -565,12 +579,14 @@ MI_API int mi_moe_gemm(const void* a_rows, int dtype, int a_stride, const void* 
       rc = 0;
       if (K >= 1024) {
         const dim3 grid((N + 7) / 8, max_tiles);
-        if (swiglu) mi::launch(moe_stream_bf16_kernel<true, 8>, grid, dim3(SW * 32), 0, stream, g);
-        else mi::launch(moe_stream_bf16_kernel<false, 8>, grid, dim3(SW * 32), 0, stream, g);
+        if (mode == GATED) mi::launch(moe_stream_bf16_kernel<GATED, 8>, grid, dim3(SW * 32), 0, stream, g);
+        else if (mode == ACTIVATED) mi::launch(moe_stream_bf16_kernel<ACTIVATED, 8>, grid, dim3(SW * 32), 0, stream, g);
+        else mi::launch(moe_stream_bf16_kernel<PLAIN, 8>, grid, dim3(SW * 32), 0, stream, g);
       } else {
         const dim3 grid((N + 15) / 16, max_tiles);
-        if (swiglu) mi::launch(moe_stream_bf16_kernel<true, 4>, grid, dim3(SW * 32), 0, stream, g);
-        else mi::launch(moe_stream_bf16_kernel<false, 4>, grid, dim3(SW * 32), 0, stream, g);
+        if (mode == GATED) mi::launch(moe_stream_bf16_kernel<GATED, 4>, grid, dim3(SW * 32), 0, stream, g);
+        else if (mode == ACTIVATED) mi::launch(moe_stream_bf16_kernel<ACTIVATED, 4>, grid, dim3(SW * 32), 0, stream, g);
+        else mi::launch(moe_stream_bf16_kernel<PLAIN, 4>, grid, dim3(SW * 32), 0, stream, g);
       }
     }
     else return mi_fail("moe_gemm: row tiles of 16 or 64 in bfloat16, got %d", TM);

@@ -255,10 +255,10 @@ MI_API int mi_rms_pair_sum(void* out, const void* a, const void* b, int dtype, c
 }
 
 // ------------------------------------------------------------------------------------------------
-// Layer norm (mean and variance, weight and bias) with the residual add in front of it.
+// Layer norm (mean and variance, weight and, optionally, bias) with the residual add in front of it.
 //
 //   sum[r, :] = resid[row(r), :] + (d1[row(r), :] + d2[row(r), :])      float32; d1, d2 optional
-//   out[r, :] = (sum - mean) * rsqrt(mean((sum - mean)^2) + eps) * w + b   rounded once to the output type
+//   out[r, :] = (sum - mean) * rsqrt(mean((sum - mean)^2) + eps) * w (+ b)   rounded once to the output type
 //   resid[row(r), :] = sum                                                 if write_back
 //
 // Two deltas because a layer whose mixer and feed-forward read the same normalised rows leaves two
@@ -298,7 +298,7 @@ __global__ void add_layernorm_kernel(TOut* __restrict__ out, float* __restrict__
   const float rstd = 1.f / sqrtf(mi::block_sum(q, scratch) / (float)H + eps);
   TOut* o = out + (size_t)r * H;
   for (int h = threadIdx.x; h < H; h += blockDim.x)
-    o[h] = mi::from_float<TOut>((ln_row[h] - mean) * rstd * w[h] + b[h]);
+    o[h] = mi::from_float<TOut>((ln_row[h] - mean) * rstd * w[h] + (b ? b[h] : 0.f));
 }
 
 
@@ -337,7 +337,7 @@ add_layernorm_vec_kernel(TOut* __restrict__ out, float* __restrict__ resid, cons
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int h = threadIdx.x + i * 256;
-    if (h < H4) { ww[i] = reinterpret_cast<const float4*>(w)[h]; bb[i] = reinterpret_cast<const float4*>(b)[h]; }
+    if (h < H4) { ww[i] = reinterpret_cast<const float4*>(w)[h]; bb[i] = b ? reinterpret_cast<const float4*>(b)[h] : make_float4(0.f, 0.f, 0.f, 0.f); }
   }
   mi::grid_dependency_sync();
   float* x = resid + (size_t)row * H;

@@ -38,7 +38,7 @@ def size_cache_pages(layer_specs, page_size: int, dtype: torch.dtype, device: to
                      utilization: float, max_num_seqs: int, max_model_len: int, max_step_tokens: Optional[int] = None) -> int:
   """Pages of a group that keeps every key, from the memory that is free now (the reference: a share of the free
   memory divided by the bytes of one token, miniinfer/utils/memory_utils.py:85-144), capped at what ``max_num_seqs``
-  requests of ``max_model_len`` tokens could ever hold.  Groups that keep a window have a size of their own
+  requests of ``max_model_len`` tokens could ever hold.  Groups that keep a window or a chunk have a size of their own
   (``KVCacheManager.group_pages``), which is taken off the memory first."""
   cap = max_num_seqs * (-(-max_model_len // page_size))
   if KVCacheManager.bytes_per_page(layer_specs, page_size, dtype) == 0:
@@ -53,7 +53,7 @@ def size_cache_pages(layer_specs, page_size: int, dtype: torch.dtype, device: to
   else:
     size = torch.empty((), dtype=dtype).element_size()
     for spec in flatten_specs(layer_specs):
-      if isinstance(spec, PagedKVSpec) and spec.window is not None:
+      if isinstance(spec, PagedKVSpec) and spec.reach is not None:
         pages = KVCacheManager.group_pages(spec, page_size, cap, max_num_seqs, max_step_tokens) + 1
         usable -= pages * 2 * spec.num_kv_heads * spec.head_dim * page_size * size
   if per_page == 0:

@@ -112,7 +112,7 @@ class Scheduler:
     # the whole request must fit the pool on its own, or it could never finish
     need = self.cache.pages_needed(None, n + req.max_tokens)
     total = [g.num_pages for g in self.cache.paged_groups]
-    windowed = [g.spec.window is not None for g in self.cache.paged_groups]
+    windowed = [g.spec.reach is not None for g in self.cache.paged_groups]
     for g, (want, have) in enumerate(zip(need, total)):
       if want > have and not windowed[g]:
         raise ValueError(f"the request needs {want} pages of cache group {g}, the pool has {have}")

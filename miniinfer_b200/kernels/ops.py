@@ -21,6 +21,7 @@ import torch
 from . import build
 
 F32, BF16 = 0, 1
+MAX_HEAD_DIM = 640   # the largest head size of the attention kernels (256 on the tensor cores)
 PREFILL_TILE = 64     # query rows of one tile of the prefill attention kernels
 PREFILL_WIDE_TILE = 128   # tokens of a work of the tcgen05 prefill kernel when a block (or each block of a pair) takes one head
 PREFILL_PAIRS_MIN_WIDE_TILES = 48   # steps with at least this many such tiles (6144 new tokens) let two blocks share a work
@@ -134,13 +135,13 @@ def embedding(out: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, scale: 
 
 
 def add_layernorm(out: torch.Tensor, resid: torch.Tensor, delta: Optional[torch.Tensor], delta2: Optional[torch.Tensor],
-                  weight: torch.Tensor, bias: torch.Tensor, eps: float, rows: Optional[torch.Tensor] = None,
+                  weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float, rows: Optional[torch.Tensor] = None,
                   write_back: bool = True) -> None:
-  """out[r] = (s - mean(s)) / sqrt(var(s) + eps) * weight + bias with s = resid[row] + (delta[row] + delta2[row]), both
+  """out[r] = (s - mean(s)) / sqrt(var(s) + eps) * weight (+ bias) with s = resid[row] + (delta[row] + delta2[row]), both
   deltas optional and of one dtype; the sum goes back to resid if write_back.  All in float32."""
   lib = common_lib()
   R, H = out.shape
-  if resid.shape[1] != H or weight.shape != (H,) or bias.shape != (H,):
+  if resid.shape[1] != H or weight.shape != (H,) or (bias is not None and bias.shape != (H,)):
     raise KernelError("add_layernorm: shapes do not match")
   for d in (delta, delta2):
     if d is not None and d.shape != resid.shape:
@@ -151,7 +152,8 @@ def add_layernorm(out: torch.Tensor, resid: torch.Tensor, delta: Optional[torch.
     raise KernelError("add_layernorm: out, rows and resid differ in rows")
   first = delta if delta is not None else delta2
   _check(lib, lib.mi_add_layernorm(_ptr(out), _dt(out), _ptr(resid, torch.float32), _ptr(delta), _ptr(delta2),
-                                   _dt(first) if first is not None else F32, _ptr(weight, torch.float32), _ptr(bias, torch.float32),
+                                   _dt(first) if first is not None else F32, _ptr(weight, torch.float32),
+                                   _ptr(bias, torch.float32) if bias is not None else _ptr(None),
                                    _ptr(rows, torch.int32) if rows is not None else _ptr(None), R, H,
                                    ctypes.c_float(eps), int(bool(write_back)), _stream()))
 
@@ -865,6 +867,50 @@ def hyper_connection(res: torch.Tensor, streams: torch.Tensor, y: Optional[torch
     _ptr(rows, torch.int32) if rows is not None else none, R, S, W, ctypes.c_float(eps), int(bool(write_back)), _stream()))
 
 
+NORM_KINDS = {"rms": 1, "layer": 2}      # what residual_step can end in
+
+
+def residual_step(out: Optional[torch.Tensor], x: torch.Tensor, y: Optional[torch.Tensor], mult: float, x_out: Optional[torch.Tensor],
+                  norm=None, rows: Optional[torch.Tensor] = None, weights: Optional[torch.Tensor] = None,
+                  first: Optional[torch.Tensor] = None, later: Optional[torch.Tensor] = None, n_later: int = 0,
+                  keep: Optional[torch.Tensor] = None) -> None:
+  """A residual stream from one sublayer to the next, float32 throughout: ``X = x + mult * y``; ``keep`` receives ``X``;
+  with ``weights [n_later + 2]`` the stream goes on as ``weights[0] first + sum_k weights[k] later[k - 1] + weights[-1] X``, else
+  as ``X``; ``x_out`` (may be ``x``) receives it, and ``out`` its norm, rounded once.  ``norm``: ``(kind, weight, bias or None, eps)`` with a
+  kind of ``NORM_KINDS``, or None (then nothing is written to ``out``).  ``x``, ``y``, ``first``, ``keep`` are ``[T, W]``, ``later [>= n_later, T, W]``;
+  ``rows``: only these rows, ``out`` holding them one after the other."""
+  lib = common_lib()
+  T, W = x.shape
+  none = _ptr(None)
+  for what, t in (("x", x), ("x_out", x_out), ("first", first), ("keep", keep)):
+    if t is not None and (t.shape != (T, W) or t.dtype != torch.float32):
+      raise KernelError(f"residual_step: {what} must be float32 {(T, W)}, got {t.dtype} {tuple(t.shape)}")
+  if y is not None and y.shape != (T, W):
+    raise KernelError(f"residual_step: the sublayer's output has shape {tuple(y.shape)}, not {(T, W)}")
+  if weights is not None and (weights.shape != (n_later + 2,) or first is None or
+                              (n_later and (later is None or later.dim() != 3 or later.shape[0] < n_later or later.shape[1:] != (T, W)
+                                            or later.dtype != torch.float32))):
+    raise KernelError("residual_step: the depth weights do not match the rows they average")
+  R = T if rows is None else rows.shape[0]
+  kind, w, b, eps = (0, None, None, 1.0) if norm is None else (NORM_KINDS[norm[0]], norm[1], norm[2], norm[3])
+  if norm is not None and (out is None or out.shape != (R, W) or w.shape != (W,) or (b is not None and b.shape != (W,))):
+    raise KernelError("residual_step: the norm's output or weights do not match")
+  dt = _dt(out) if out is not None else (_dt(y) if y is not None else F32)
+  _check(lib, lib.mi_residual_step(
+    _ptr(out) if out is not None else none, dt, _ptr(x), _ptr(y) if y is not None else none, _dt(y) if y is not None else dt,
+    ctypes.c_float(mult), _ptr(keep) if keep is not None else none, _ptr(x_out) if x_out is not None else none,
+    _ptr(weights, torch.float32) if weights is not None else none, _ptr(first) if first is not None else none,
+    _ptr(later) if (later is not None and n_later) else none, ctypes.c_longlong(T * W), int(n_later) if weights is not None else 0, kind,
+    _ptr(w, torch.float32) if w is not None else none, _ptr(b, torch.float32) if b is not None else none, ctypes.c_float(eps),
+    _ptr(rows, torch.int32) if rows is not None else none, R, W, _stream()))
+
+
+def softcap(x: torch.Tensor, cap: float) -> None:
+  """x <- cap * tanh(x / cap), float32, in place."""
+  lib = common_lib()
+  _check(lib, lib.mi_softcap(_ptr(x, torch.float32), ctypes.c_longlong(x.numel()), ctypes.c_float(cap), _stream()))
+
+
 def relu_squared(out: torch.Tensor, x: torch.Tensor) -> None:
   """out = max(x, 0)^2 element by element, squared in float32 and rounded once; ``out`` may be ``x``."""
   lib = common_lib()
@@ -974,7 +1020,7 @@ def _glu(kind: str, limit: float):
 
 def routed_experts(out: torch.Tensor, x: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], gate_up: torch.Tensor,
                    down: torch.Tensor, top: int, workspace, weights: str = "sigmoid_share", glu: str = "silu", limit: float = 0.0,
-                   shared: Optional[torch.Tensor] = None, shared_gated: bool = False) -> None:
+                   shared: Optional[torch.Tensor] = None, shared_gated: bool = False, weight_scale: float = 1.0) -> None:
   """out[t] = sum over the ``top`` chosen experts of weight * down_e(silu(gate_e x) * up_e x).
 
   ``router [E, H]`` in the rows' dtype and ``correction [E]`` float32: logits ``router x`` accumulated in float32 (bfloat16
@@ -987,19 +1033,23 @@ def routed_experts(out: torch.Tensor, x: torch.Tensor, router: torch.Tensor, cor
   softmax over the chosen logits alone.  ``glu``/``limit``: the experts' gated activation (``silu``, or ``clamped`` with its
   limit: ``g' = min(g, L)``, ``u' = clamp(u, -L, L)``, ``g' sigmoid(1.702 g') (u' + 1)``).  ``shared [T, H]``: the output of an
   expert that every token runs through, added to the sum; with ``shared_gated`` the router has one row more than there are
-  experts, and the shared rows are multiplied with the sigmoid of that row's logit, one number a token."""
+  experts, and the shared rows are multiplied with the sigmoid of that row's logit, one number a token.
+
+  ``glu="relu_squared"``: experts without a gate, ``gate_up [E, ff, H]`` holding their up rows alone: ``down_e(max(up_e x, 0)^2)``.
+  ``weight_scale``: a constant the experts' weights are multiplied with."""
   lib = common_lib()
   T, H = x.shape
   E = router.shape[0] - (1 if shared_gated else 0)
   ff = down.shape[2]
-  if weights not in ("sigmoid_share", "softmax_chosen") or (correction is None and weights == "sigmoid_share"):
-    raise KernelError(f"routed_experts: weights={weights!r} is not known, or sigmoid shares without their correction")
+  if weights not in ("sigmoid_share", "softmax_chosen"):
+    raise KernelError(f"routed_experts: weights={weights!r} is not known")
   if shared_gated and shared is None:
     raise KernelError("routed_experts: a gate for the shared expert without its rows")
   if shared is not None and (shared.shape != (T, H) or shared.dtype != out.dtype or not shared.is_contiguous()):
     raise KernelError("routed_experts: the shared expert's rows do not match the output")
-  kind, lim = _glu(glu, limit)
-  if router.shape != (E + (1 if shared_gated else 0), H) or (correction is not None and correction.shape != (E,)) or gate_up.shape != (E, 2 * ff, H) or down.shape != (E, H, ff) or out.shape != (T, H):
+  gated = glu != "relu_squared"
+  kind, lim = _glu(glu, limit) if gated else (0, ctypes.c_float(0.0))
+  if router.shape != (E + (1 if shared_gated else 0), H) or (correction is not None and correction.shape != (E,)) or gate_up.shape != (E, (2 if gated else 1) * ff, H) or down.shape != (E, H, ff) or out.shape != (T, H):
     raise KernelError(f"routed_experts: shapes do not match: x {tuple(x.shape)}, router {tuple(router.shape)}, "
                       f"gate_up {tuple(gate_up.shape)}, down {tuple(down.shape)}")
   if gate_up.dtype != x.dtype or down.dtype != x.dtype or out.dtype != x.dtype or router.dtype != x.dtype:
@@ -1027,7 +1077,7 @@ def routed_experts(out: torch.Tensor, x: torch.Tensor, router: torch.Tensor, cor
   logits = workspace.buffer("moe_logits", (T, Z), torch.float32)
   linear(logits, x, router)
   _check(lib, lib.mi_moe_route(_ptr(logits, torch.float32), Z, T, _ptr(correction, torch.float32) if correction is not None else _ptr(None), E, top,
-                               1 if weights == "softmax_chosen" else 0, _ptr(idx), _ptr(wts), st))
+                               1 if weights == "softmax_chosen" else 0, ctypes.c_float(weight_scale), _ptr(idx), _ptr(wts), st))
   shared_args = (_ptr(shared) if shared is not None else _ptr(None),
                  ctypes.c_void_p(logits.data_ptr() + 4 * E) if shared_gated else _ptr(None), Z)
   _check(lib, lib.mi_moe_align(_ptr(idx), pairs, E, tile, _ptr(sorted_pair), _ptr(pos_of), _ptr(tile_expert), rows, tiles, st))
@@ -1036,13 +1086,13 @@ def routed_experts(out: torch.Tensor, x: torch.Tensor, router: torch.Tensor, cor
     y16 = workspace.buffer("moe_y16", (rows, H), x.dtype)
     status = workspace.zeros("gemm_tc_status", 1, torch.int32)
     _check(lib, lib.mi_moe_gather(_ptr(xs), _ptr(x), _ptr(sorted_pair), rows, top, H, st))
-    _check(lib, lib.mi_gemm_tc_grouped_bf16(_ptr(act), _ptr(xs), _ptr(gate_up), rows, ff, H, ff, E, 1, _ptr(tile_expert), tile,
-                                            _ptr(status, torch.int32), _tc_pairs(), kind, lim, st))
+    _check(lib, lib.mi_gemm_tc_grouped_bf16(_ptr(act), _ptr(xs), _ptr(gate_up), rows, ff, H, ff, E, int(gated), _ptr(tile_expert), tile,
+                                            _ptr(status, torch.int32), _tc_pairs(), kind, lim, int(not gated), st))
     _check(lib, lib.mi_gemm_tc_grouped_bf16(_ptr(y16), _ptr(act), _ptr(down), rows, H, ff, H, E, 0, _ptr(tile_expert), tile,
-                                            _ptr(status, torch.int32), _tc_pairs(), 0, ctypes.c_float(0.0), st))
+                                            _ptr(status, torch.int32), _tc_pairs(), 0, ctypes.c_float(0.0), 0, st))
     _check(lib, lib.mi_moe_combine(_ptr(out), _dt(out), _ptr(y16), BF16, _ptr(pos_of), _ptr(wts), T, top, H, *shared_args, st))
     return
-  _check(lib, lib.mi_moe_gemm(_ptr(x), dt, H, _ptr(gate_up), _ptr(act), _ptr(sorted_pair), _ptr(tile_expert), tiles, tile, ff, H, top, 1, kind, lim, st))
+  _check(lib, lib.mi_moe_gemm(_ptr(x), dt, H, _ptr(gate_up), _ptr(act), _ptr(sorted_pair), _ptr(tile_expert), tiles, tile, ff, H, top, 1 if gated else 2, kind, lim, st))
   _check(lib, lib.mi_moe_gemm(_ptr(act), dt, ff, _ptr(down), _ptr(y), _ptr(sorted_pair), _ptr(tile_expert), tiles, tile, H, ff, top, 0, 0,
                               ctypes.c_float(0.0), st))
   _check(lib, lib.mi_moe_combine(_ptr(out), _dt(out), _ptr(y), F32, _ptr(pos_of), _ptr(wts), T, top, H, *shared_args, st))
@@ -1204,7 +1254,8 @@ def attention(out: torch.Tensor, qkv: torch.Tensor, kv_layer: torch.Tensor, bloc
               batch: AttentionBatch, num_heads: int, num_kv_heads: int, head_dim: int, scale: float,
               window: Optional[int], force_generic: bool = False, sink: Optional[torch.Tensor] = None,
               gate: Optional[torch.Tensor] = None, gate_offset: int = 0, out_hd: Optional[int] = None,
-              keep_first: int = 0, softcap: float = 0.0, score_bias: Optional[torch.Tensor] = None) -> None:
+              keep_first: int = 0, softcap: float = 0.0, score_bias: Optional[torch.Tensor] = None,
+              chunk: Optional[int] = None, gate_per_head: bool = False, distance: Optional[torch.Tensor] = None) -> None:
   """out[t, h*hd:(h+1)*hd] = softmax(scale * q . K^T over the keys the token may see) V, reading
   K and V through the block table.  ``qkv`` holds the step's fused rows; q is its first part.
 
@@ -1214,7 +1265,10 @@ def attention(out: torch.Tensor, qkv: torch.Tensor, kv_layer: torch.Tensor, bloc
   ``out_hd`` values of each head are written, ``out`` being ``[tokens, heads * out_hd]`` (cache rows padded to ``head_dim``);
   ``keep_first`` - with a window, every token also sees the first ``keep_first`` keys of its request; ``softcap`` > 0 - a
   scaled score ``s`` becomes ``softcap * tanh(s / softcap)``; ``score_bias [heads]`` float32 - no softmax: the weight of a
-  visible key is ``sigmoid(s + score_bias[head])``, not normalised over the keys (no sink then)."""
+  visible key is ``sigmoid(s + score_bias[head])``, not normalised over the keys (no sink then); ``chunk`` - a token sees
+  the keys of its own chunk of that many positions only, chunks being counted from position 0 (not with a window);
+  ``gate_per_head`` - the gate's columns are one per head, not one per value; ``distance [2 * heads]`` float32, all r1 and
+  then all r2 - a softmax score loses ``r1[head] * ln(1 + r2[head] * (i - j))``."""
   T = qkv.shape[0]
   ohd = head_dim if out_hd is None else int(out_hd)
   if out.shape != (T, num_heads * ohd) or out.dtype != qkv.dtype or kv_layer.dtype != qkv.dtype or not (0 < ohd <= head_dim):
@@ -1227,17 +1281,24 @@ def attention(out: torch.Tensor, qkv: torch.Tensor, kv_layer: torch.Tensor, bloc
   gate_stride = 0
   if gate is not None:
     gate_stride = gate.shape[1]
-    if gate.dtype != qkv.dtype or gate.shape[0] != T or gate_offset + num_heads * ohd > gate_stride or not gate.is_contiguous():
+    gate_width = num_heads * (1 if gate_per_head else ohd)
+    if gate.dtype != qkv.dtype or gate.shape[0] != T or gate_offset + gate_width > gate_stride or not gate.is_contiguous():
       raise KernelError("attention: the gate rows do not match")
   if score_bias is not None and (score_bias.shape != (num_heads,) or score_bias.dtype != torch.float32 or sink is not None):
     raise KernelError("attention: the score biases must be one float32 per query head, and go without sinks")
   if softcap < 0:
     raise KernelError(f"attention: softcap={softcap} must not be negative")
+  if distance is not None and (distance.shape != (2 * num_heads,) or distance.dtype != torch.float32 or score_bias is not None):
+    raise KernelError("attention: the distance biases must be two float32 per query head, and go with a softmax")
+  if chunk and window:
+    raise KernelError("attention: a window and chunks exclude each other")
   opts = _AttentionOptions(sink, gate, gate_offset, gate_stride, ohd)
   opts.softcap, opts.score_bias = float(softcap), score_bias
-  win = int(window) if window else 0
-  opts.keep_first = int(keep_first) if win else 0
-  even = ohd % 2 == 0 and gate_offset % 2 == 0 and gate_stride % 2 == 0
+  opts.gate_per_head, opts.distance = bool(gate_per_head), distance
+  # the kernels take what a token sees as one number: a window, or the negated chunk size, or 0 for every earlier key
+  win = int(window) if window else (-int(chunk) if chunk else 0)
+  opts.keep_first = int(keep_first) if win > 0 else 0
+  even = ohd % 2 == 0 and (gate_per_head or (gate_offset % 2 == 0 and gate_stride % 2 == 0))
   if qkv.dtype == torch.bfloat16 and not force_generic and head_dim % 16 == 0 and 16 <= head_dim <= 256 and even:
     _attention_bf16(out, qkv, kv_layer, block_table, batch, num_heads, num_kv_heads, head_dim, scale, win, page_size, opts)
     return
@@ -1247,21 +1308,22 @@ def attention(out: torch.Tensor, qkv: torch.Tensor, kv_layer: torch.Tensor, bloc
     block_table.shape[1], _ptr(batch.token_item, torch.int32), _ptr(batch.positions, torch.int32),
     _ptr(batch.seq_slot, torch.int32), T, num_heads, num_kv_heads, head_dim, page_size,
     ctypes.c_float(scale), win, opts.sink_ptr(), opts.gate_ptr(), gate_stride, ohd, opts.keep_first, ctypes.c_float(opts.softcap),
-    opts.score_bias_ptr(), _stream()))
+    opts.score_bias_ptr(), int(opts.gate_per_head), opts.distance_ptr(), _stream()))
 
 
 class _AttentionOptions:
   """The optional sink, output gate and output width of an attention call, as the kernels take them."""
 
-  __slots__ = ("sink", "gate", "gate_offset", "gate_stride", "out_hd", "keep_first", "softcap", "score_bias")
+  __slots__ = ("sink", "gate", "gate_offset", "gate_stride", "out_hd", "keep_first", "softcap", "score_bias", "gate_per_head", "distance")
 
   def __init__(self, sink, gate, gate_offset, gate_stride, out_hd, keep_first=0):
     self.sink, self.gate, self.gate_offset, self.gate_stride, self.out_hd = sink, gate, gate_offset, gate_stride, out_hd
     self.keep_first = keep_first
     self.softcap, self.score_bias = 0.0, None
+    self.gate_per_head, self.distance = False, None
 
-  def shaped_scores(self) -> bool:
-    return self.softcap > 0 or self.score_bias is not None
+  def distance_ptr(self):
+    return _ptr(self.distance, torch.float32) if self.distance is not None else _ptr(None)
 
   def score_bias_ptr(self):
     return _ptr(self.score_bias, torch.float32) if self.score_bias is not None else _ptr(None)
@@ -1394,7 +1456,7 @@ def _attention_bf16(out, qkv, kv_layer, block_table, batch, nh, nkv, hd, scale, 
   whole_heads = opts.out_hd == hd and not opts.keep_first
   if batch.num_prefill_tiles:
     # the tcgen05 kernel takes sink and gate; its output rows are whole heads, and it reads the gate 16 bytes at a time
-    gate_ok = opts.gate is None or (opts.gate_offset % 8 == 0 and opts.gate_stride % 8 == 0 and opts.gate.data_ptr() % 16 == 0)
+    gate_ok = opts.gate is None or opts.gate_per_head or (opts.gate_offset % 8 == 0 and opts.gate_stride % 8 == 0 and opts.gate.data_ptr() % 16 == 0)
     use_tc = (opts.out_hd == hd and gate_ok and page_size % 64 == 0 and lib.mi_attention_prefill_tc_supported() == 1
               and os.environ.get("MINIINFER_B200_PREFILL_TC", "1") != "0")
     if use_tc:
@@ -1413,7 +1475,8 @@ def _attention_bf16(out, qkv, kv_layer, block_table, batch, nh, nkv, hd, scale, 
         _ptr(batch.q_len, torch.int32), _ptr(batch.ctx_len, torch.int32), _ptr(batch.seq_slot, torch.int32),
         _ptr(status, torch.int32), nh, nkv, page_size, ctypes.c_float(scale), win, _num_sms(qkv.device), _stream(),
         _ptr(wide, torch.int32) if wide is not None else _ptr(None), n_wide, pairs,
-        opts.sink_ptr(), opts.gate_ptr(), opts.gate_stride, opts.keep_first, ctypes.c_float(opts.softcap), opts.score_bias_ptr()))
+        opts.sink_ptr(), opts.gate_ptr(), opts.gate_stride, opts.keep_first, ctypes.c_float(opts.softcap), opts.score_bias_ptr(),
+        int(opts.gate_per_head), opts.distance_ptr()))
       if batch.scratch is None and int(status[0]) != 0:
         raise KernelError("attention_prefill_tc: a bounded wait on a barrier ran out")
     else:
@@ -1422,13 +1485,13 @@ def _attention_bf16(out, qkv, kv_layer, block_table, batch, nh, nkv, hd, scale, 
         _ptr(batch.prefill_tiles, torch.int32), batch.num_prefill_tiles, _ptr(batch.q_start, torch.int32),
         _ptr(batch.q_len, torch.int32), _ptr(batch.ctx_len, torch.int32), _ptr(batch.seq_slot, torch.int32),
         nh, nkv, page_size, ctypes.c_float(scale), win, opts.sink_ptr(), opts.gate_ptr(), opts.gate_stride, opts.out_hd,
-        opts.keep_first, ctypes.c_float(opts.softcap), opts.score_bias_ptr(), _stream()))
+        opts.keep_first, ctypes.c_float(opts.softcap), opts.score_bias_ptr(), int(opts.gate_per_head), opts.distance_ptr(), _stream()))
   if batch.num_decode:
-    span = min(batch.max_ctx_len, win) if win else batch.max_ctx_len
+    span = min(batch.max_ctx_len, abs(win)) if win else batch.max_ctx_len      # the most keys a token sees
     G = nh // nkv
     tma_shapes = whole_heads and hd % 64 == 0 and page_size % 64 == 0 and os.environ.get("MINIINFER_B200_DECODE_TMA", "1") != "0"
-    # shaped scores (a cap, sigmoid weights) the persistent TMA kernel and the cp.async kernel know, the cluster kernel does not
-    cluster = decode_cluster_size(lib, hd, batch.num_decode, nkv, span) if (tma_shapes and G <= 8 and not opts.shaped_scores()) else 0
+    # sigmoid weights the persistent TMA kernel and the cp.async kernel know, the cluster kernel does not
+    cluster = decode_cluster_size(lib, hd, batch.num_decode, nkv, span) if (tma_shapes and G <= 8 and opts.score_bias is None) else 0
     if cluster:
       if batch.scratch is not None:
         status = batch.scratch.zeros("attention_decode_counters", batch.num_decode * nkv + 1, torch.int32)[:1]
@@ -1438,7 +1501,8 @@ def _attention_bf16(out, qkv, kv_layer, block_table, batch, nh, nkv, hd, scale, 
         _ptr(out), _ptr(qkv), qkv.shape[1], _kv_tensor_map(lib, kv_layer), _ptr(block_table, torch.int32), block_table.shape[1],
         _ptr(batch.decode_items, torch.int32), _ptr(batch.q_start, torch.int32), _ptr(batch.ctx_len, torch.int32),
         _ptr(batch.seq_slot, torch.int32), _ptr(status, torch.int32), batch.num_decode, nh, nkv, page_size, ctypes.c_float(scale), win,
-        cluster, batch.max_ctx_len, _stream(), opts.sink_ptr(), opts.gate_ptr(), opts.gate_stride))
+        cluster, batch.max_ctx_len, _stream(), opts.sink_ptr(), opts.gate_ptr(), opts.gate_stride, int(opts.gate_per_head),
+        ctypes.c_float(opts.softcap), opts.distance_ptr()))
       if batch.scratch is None and int(status[0]) != 0:
         raise KernelError("attention_decode_cluster: a bounded wait on a copy barrier ran out")
       return
@@ -1466,7 +1530,8 @@ def _attention_bf16(out, qkv, kv_layer, block_table, batch, nh, nkv, hd, scale, 
         _ptr(batch.decode_items, torch.int32), _ptr(batch.q_start, torch.int32), _ptr(batch.ctx_len, torch.int32),
         _ptr(batch.seq_slot, torch.int32), _ptr(scratch, torch.float32), _ptr(counters[1:], torch.int32), _ptr(counters[:1], torch.int32),
         batch.num_decode, nh, nkv, page_size, ctypes.c_float(scale), win, chunk, max_splits, _num_sms(qkv.device), _stream(),
-        opts.sink_ptr(), opts.gate_ptr(), opts.gate_stride, ctypes.c_float(opts.softcap), opts.score_bias_ptr()))
+        opts.sink_ptr(), opts.gate_ptr(), opts.gate_stride, ctypes.c_float(opts.softcap), opts.score_bias_ptr(),
+        int(opts.gate_per_head), opts.distance_ptr()))
       if batch.scratch is None and int(counters[0]) != 0:
         raise KernelError("attention_decode_tma: a bounded wait on a copy barrier ran out")
     else:
@@ -1476,7 +1541,7 @@ def _attention_bf16(out, qkv, kv_layer, block_table, batch, nh, nkv, hd, scale, 
         _ptr(batch.seq_slot, torch.int32), _ptr(scratch, torch.float32), _ptr(counters[1:], torch.int32),
         batch.num_decode, nh, nkv, page_size, ctypes.c_float(scale), win, chunk, max_splits,
         opts.sink_ptr(), opts.gate_ptr(), opts.gate_stride, opts.out_hd, opts.keep_first, ctypes.c_float(opts.softcap),
-        opts.score_bias_ptr(), _stream()))
+        opts.score_bias_ptr(), int(opts.gate_per_head), opts.distance_ptr(), _stream()))
 
 
 _tensor_maps: Dict[tuple, ctypes.Array] = {}

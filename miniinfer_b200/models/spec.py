@@ -68,8 +68,8 @@ class ModelSpec:
 
     for b in self.blocks:
       walk(b)
-    out.append(self.final_norm)
-    out.append(self.lm_head)
+    walk(self.final_norm)
+    walk(self.lm_head)
     return out
 
   def cache_layer_specs(self) -> List[Optional[CacheSpec]]:

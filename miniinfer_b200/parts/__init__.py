@@ -1,6 +1,7 @@
 from .base import (Block, Embedding, FeedForward, Head, HostStep, Mixer, Norm, ParamSpec, Part, Piece, PositionEncoding,
                    StepWork, whole)
 from .block import OutputNormBlock, ParallelBlock, PreNormBlock
+from .depth import DepthAverageBlock, DepthAverageNorm
 from .embedding import LMHead, TokenEmbedding
 from .feedforward import ActivatedFeedForward, RoutedExpertsFeedForward, SwiGLUFeedForward
 from .gated_attention import GatedAttentionMixer
@@ -30,6 +31,7 @@ register_feed_forward("activated")(ActivatedFeedForward)
 register_norm("rmsnorm")(RMSNorm)
 register_norm("layernorm")(LayerNorm)
 register_norm("stream_sum_rmsnorm")(StreamSumNorm)
+register_norm("depth_average")(DepthAverageNorm)
 register_position_encoding("rotary")(RotaryEncoding)
 register_position_encoding("scaled_rotary")(ScaledRotaryEncoding)
 register_position_encoding("band_scaled_rotary")(BandScaledRotaryEncoding)
@@ -37,3 +39,4 @@ register_block("pre_norm")(PreNormBlock)
 register_block("parallel")(ParallelBlock)
 register_block("hyper_connection")(HyperConnectionBlock)
 register_block("output_norm")(OutputNormBlock)
+register_block("depth_average")(DepthAverageBlock)

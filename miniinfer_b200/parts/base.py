@@ -158,6 +158,12 @@ class Norm(Part):
     that follows it may then compute itself (``takes_residual``); None otherwise."""
     return None
 
+  def as_row_norm(self):
+    """(kind, weight, bias or None, eps) if this norm is one of ``ops.NORM_KINDS`` over a row, for blocks whose own kernel
+    ends in the norm; None otherwise."""
+    rms = self.as_rms()
+    return None if rms is None else ("rms", rms[0], None, rms[1])
+
   def add_norm(self, resid: torch.Tensor, delta: Optional[torch.Tensor], ctx) -> torch.Tensor:
     raise NotImplementedError
 

@@ -48,12 +48,17 @@ class TokenEmbedding(Embedding):
 
 
 class LMHead(Head):
+  """``softcap`` > 0: the logits leave as ``softcap * tanh(logits / softcap)``."""
+
   def __init__(self, name: str, vocab_size: int, hidden_size: int, tied_to: Optional[TokenEmbedding] = None,
-               tensor: Optional[str] = None):
+               tensor: Optional[str] = None, softcap: float = 0.0):
     super().__init__(name)
+    if not softcap >= 0:
+      raise ValueError(f"{name}: softcap must not be negative, got {softcap!r}")
     self.vocab_size = vocab_size
     self.hidden_size = hidden_size
     self.tied_to = tied_to
+    self.softcap = float(softcap)
     self.tensor = tensor or f"{name}.weight"
 
   def param_specs(self) -> Dict[str, ParamSpec]:
@@ -73,4 +78,6 @@ class LMHead(Head):
   def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
     out = ctx.ws.buffer("logits", (x.shape[0], self.vocab_size), torch.float32)
     ops.linear(out, x, self.table())
+    if self.softcap > 0:
+      ops.softcap(out, self.softcap)
     return out

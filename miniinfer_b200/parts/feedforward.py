@@ -13,11 +13,16 @@ from .base import FeedForward, ParamSpec, Piece, whole
 
 
 class SwiGLUFeedForward(FeedForward):
-  """``tensors``: the file names of the gate, up and down matrices after ``<name>.`` (default: ``gate_proj.weight``,
+  """``activation``: ``silu``, or ``clamped`` with its ``limit``: ``g = min(gate x, limit)``, ``u = clamp(up x, -limit, limit)``,
+  ``g * sigmoid(1.702 g) * (u + 1)`` in place of ``silu(gate x) * up x``.  ``tensors``: the file names of the gate, up and down matrices after ``<name>.`` (default: ``gate_proj.weight``,
   ``up_proj.weight``, ``down_proj.weight``, with ``gate_up_proj.weight`` accepted for the fused pair)."""
 
-  def __init__(self, name: str, hidden_size: int, intermediate_size: int, tensors: Optional[Tuple[str, str, str]] = None):
+  def __init__(self, name: str, hidden_size: int, intermediate_size: int, tensors: Optional[Tuple[str, str, str]] = None,
+               activation: str = "silu", limit: float = 0.0):
     super().__init__(name)
+    if activation not in ops.GLU_KINDS or (activation == "clamped" and not limit > 0):
+      raise ValueError(f"{name}: activation={activation!r} is not known ({', '.join(ops.GLU_KINDS)}) or its limit {limit!r} is not positive")
+    self.activation, self.limit = activation, float(limit)
     self.hidden_size = hidden_size
     self.intermediate_size = intermediate_size
     self.tensors = tensors
@@ -43,7 +48,7 @@ class SwiGLUFeedForward(FeedForward):
           raise ValueError(f"{self.name}: {what}={k} must be a multiple of 8 in bfloat16 (rows are read 16 bytes at a time)")
 
   def takes_residual(self, norm, ctx) -> bool:
-    return norm.as_rms() is not None and ops.fuses_few_rows(ctx.num_tokens, ctx.dtype)
+    return self.activation == "silu" and norm.as_rms() is not None and ops.fuses_few_rows(ctx.num_tokens, ctx.dtype)
 
   def forward_on_residual(self, resid: torch.Tensor, norm, ctx) -> None:
     """Two kernels: norm + gate-and-up product + SwiGLU, then the down product + residual add."""
@@ -55,7 +60,7 @@ class SwiGLUFeedForward(FeedForward):
   def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
     T = x.shape[0]
     act = ctx.ws.buffer("ffn_act", (T, self.intermediate_size), ctx.dtype)
-    ops.linear_swiglu(act, x, self.gate_up, ctx.ws)
+    ops.linear_glu(act, x, self.gate_up, ctx.ws, self.activation, self.limit)
     out = ctx.ws.buffer("ffn_out", (T, self.hidden_size), ctx.dtype)
     ops.linear(out, act, self.down)
     return out
@@ -98,36 +103,41 @@ class ActivatedFeedForward(FeedForward):
 
 
 class RoutedExpertsFeedForward(FeedForward):
-  """A mixture of ``num_experts`` small gated feed-forward layers of which each token uses ``top``.
+  """A mixture of ``num_experts`` small feed-forward layers of which each token uses ``top``.
 
   Router logits ``z = W_router h`` accumulated in float32 by the engine's matrix product (in bfloat16 mode both operands
   are bfloat16, whose products are exact in float32).  ``router_weights="sigmoid_share"``: scores ``s = sigmoid(z)`` in float32;
   the experts of the ``top`` largest ``s + correction`` are chosen; their weights are their ``s`` (without the correction)
-  divided by the sum of those ``s`` (+ 1e-20).  ``router_weights="softmax_chosen"``: the ``top`` largest logits are chosen, the
-  weights are the softmax over the chosen logits alone, and there is no correction.  The output is the weighted sum of the
+  divided by the sum of those ``s`` (+ 1e-20).  ``correction`` False: there is none, and the largest scores are chosen.
+  ``router_weights="softmax_chosen"``: the ``top`` largest logits are chosen, the
+  weights are the softmax over the chosen logits alone, and there is no correction.  ``weight_scale``: a constant that
+  multiplies the weights.  The output is the weighted sum of the
   chosen experts' outputs.
 
   An expert is ``down(act(gate x) * up x)`` with ``activation="silu"`` or ``activation="clamped"`` and its ``limit``:
-  ``g = min(gate x, limit)``, ``u = clamp(up x, -limit, limit)``, ``g * sigmoid(1.702 g) * (u + 1)``.
+  ``g = min(gate x, limit)``, ``u = clamp(up x, -limit, limit)``, ``g * sigmoid(1.702 g) * (u + 1)``.  With ``activation="relu_squared"`` it has no gate: ``down(max(up x, 0)^2)``.
 
   ``shared_size``: an expert of that size more (``shared_limit`` its limit, same form) that every token runs through; its
   output is added to the sum, times ``sigmoid(w_sg . h)`` - one number a token - if ``shared_gate``.  The gate's row rides as
   the last row of the router's matrix, so its logit comes out of the router's product.
 
-  The experts' matrices are stacked: ``gate_up [E, 2 ff, H]`` (an expert's gate rows, then its up rows), ``down [E, H, ff]``.
+  The experts' matrices are stacked: ``gate_up [E, 2 ff, H]`` (an expert's gate rows, then its up rows; without a gate
+  ``[E, ff, H]``), ``down [E, H, ff]``.
   File tensors: ``<name>.router``, ``<name>.correction``, ``<name>.e<i>.gate`` / ``.up`` / ``.down``,
   ``<name>.shared.gate`` / ``.up`` / ``.down`` / ``.sg``."""
 
   def __init__(self, name: str, hidden_size: int, expert_size: int, num_experts: int, top: int, router_weights: str = "sigmoid_share",
                activation: str = "silu", limit: float = 0.0, shared_size: Optional[int] = None, shared_limit: Optional[float] = None,
-               shared_gate: bool = False):
+               shared_gate: bool = False, correction: bool = True, weight_scale: float = 1.0):
     super().__init__(name)
     if not (1 <= top <= num_experts):
       raise ValueError(f"{name}: top={top} must lie in 1..experts={num_experts}")
     if router_weights not in ("sigmoid_share", "softmax_chosen"):
       raise ValueError(f"{name}: router_weights={router_weights!r} is not known (sigmoid_share, softmax_chosen)")
-    if activation not in ops.GLU_KINDS or (activation == "clamped" and not limit > 0):
-      raise ValueError(f"{name}: activation={activation!r} is not known ({', '.join(ops.GLU_KINDS)}) or its limit {limit!r} is not positive")
+    if (activation not in ops.GLU_KINDS and activation != "relu_squared") or (activation == "clamped" and not limit > 0):
+      raise ValueError(f"{name}: activation={activation!r} is not known ({', '.join(ops.GLU_KINDS)}, relu_squared) or its limit {limit!r} is not positive")
+    if activation == "relu_squared" and shared_size is not None:
+      raise ValueError(f"{name}: a shared expert has a gate, the experts of {activation!r} have none")
     if shared_size is None and shared_gate:
       raise ValueError(f"{name}: a gate for a shared expert that is not there")
     if shared_size is not None and shared_size <= 0:
@@ -137,6 +147,9 @@ class RoutedExpertsFeedForward(FeedForward):
     self.num_experts = num_experts
     self.top = top
     self.router_weights = router_weights
+    self.has_correction = bool(correction) and router_weights == "sigmoid_share"
+    self.weight_scale = float(weight_scale)
+    self.gated = activation != "relu_squared"
     self.activation, self.limit = activation, float(limit)
     self.shared_size = shared_size
     self.shared_limit = float(shared_limit) if shared_limit is not None else float(limit)
@@ -146,15 +159,18 @@ class RoutedExpertsFeedForward(FeedForward):
 
   def param_specs(self) -> Dict[str, ParamSpec]:
     H, F, E, n = self.hidden_size, self.expert_size, self.num_experts, self.name
-    gate_up = [p for e in range(E) for p in (Piece(f"{n}.e{e}.gate", 2 * F * e, (F, H)), Piece(f"{n}.e{e}.up", 2 * F * e + F, (F, H)))]
+    if self.gated:
+      gate_up = [p for e in range(E) for p in (Piece(f"{n}.e{e}.gate", 2 * F * e, (F, H)), Piece(f"{n}.e{e}.up", 2 * F * e + F, (F, H)))]
+    else:
+      gate_up = [Piece(f"{n}.e{e}.up", F * e, (F, H)) for e in range(E)]
     down = [Piece(f"{n}.e{e}.down", H * e, (H, F)) for e in range(E)]
     router = [Piece(f"{n}.router", 0, (E, H))] + ([Piece(f"{n}.shared.sg", E, (1, H))] if self.shared_gate else [])
     specs = {
       "router": ParamSpec((E + (1 if self.shared_gate else 0), H), "matrix", [router], init="fan_in"),
-      "gate_up": ParamSpec((2 * F * E, H), "matrix", [gate_up]),
+      "gate_up": ParamSpec(((2 if self.gated else 1) * F * E, H), "matrix", [gate_up]),
       "down": ParamSpec((H * E, F), "matrix", [down]),
     }
-    if self.router_weights == "sigmoid_share":
+    if self.has_correction:
       specs["correction"] = ParamSpec((E,), "vector", [whole(f"{n}.correction", (E,))])
     if self.shared_size is not None:
       S = self.shared_size
@@ -180,7 +196,8 @@ class RoutedExpertsFeedForward(FeedForward):
       shared = ctx.ws.buffer("ffn_shared", (T, H), ctx.dtype)
       ops.linear(shared, act, self.shared_down)
     out = ctx.ws.buffer("ffn_out", (T, H), ctx.dtype)
-    ops.routed_experts(out, x, self.router, self.correction if self.router_weights == "sigmoid_share" else None,
-                       self.gate_up.view(E, 2 * F, H), self.down.view(E, H, F), self.top, ctx.ws, weights=self.router_weights,
-                       glu=self.activation, limit=self.limit, shared=shared, shared_gated=self.shared_gate)
+    ops.routed_experts(out, x, self.router, self.correction if self.has_correction else None,
+                       self.gate_up.view(E, (2 if self.gated else 1) * F, H), self.down.view(E, H, F), self.top, ctx.ws, weights=self.router_weights,
+                       glu=self.activation, limit=self.limit, shared=shared, shared_gated=self.shared_gate,
+                       weight_scale=self.weight_scale)
     return out

@@ -18,13 +18,17 @@ key/value head ``i // (H / G)``), query/key size ``dim`` and value size ``vdim``
     values that the layer with ``value_mix="source"`` made for the same token in this step (handed on through
     ``ctx.shared[value_mix_key]``); what is cached is the mixed ``v`` and the normalised ``k``;
   * token ``i`` sees token ``j`` of its request if ``0 <= i - j < window`` (``window`` None: every earlier token) or, with
-    ``keep_first``, if ``j < keep_first`` and ``j <= i``: the first tokens stay visible, at their true positions;
+    ``keep_first``, if ``j < keep_first`` and ``j <= i``: the first tokens stay visible, at their true positions; with ``chunk``
+    it sees the earlier tokens of its own chunk, ``floor(i / chunk) == floor(j / chunk)``, positions counted in the request;
+  * ``distance_bias``: a scaled score loses ``r1 * ln(1 + r2 * (i - j))``, two learned numbers per query head (file tensors
+    ``r1``, ``r2``);
   * ``softmax`` over ``scale * q . k`` whose denominator also holds ``exp(sink)`` of the query head (``sinks``), a term
     with no key and no value;
   * ``softcap`` > 0: a scaled score ``s`` becomes ``softcap * tanh(s / softcap)`` before the weights are made;
   * ``weights="sigmoid"``: no softmax - the weight of a visible key is ``sigmoid(s + b)`` with ``b`` a learned number per
     query head (file tensor ``pb``), and the weights are not normalised over the keys (``sinks`` must be off);
-  * the heads' outputs, side by side, are multiplied element by element with ``sigmoid(g)`` (``gated``), then projected.
+  * the heads' outputs, side by side, are multiplied element by element with ``sigmoid(g)`` (``gated``) - or, with
+    ``gate_per_head``, every head's output with the sigmoid of one number of its own -, then projected.
 
 Every option can be switched off, so other designs may take the parts they need.  The cache keeps keys and values in
 rows of one size, ``max(dim, vdim)`` rounded up to a multiple of 16 and zero-filled: a zero tail adds nothing to a score,
@@ -49,7 +53,8 @@ class GatedAttentionMixer(AttentionMixer):
                value_mix: Optional[str] = None, value_mix_key: str = "value_mix_source",
                tensors: Optional[Dict[str, str]] = None, rotary: Optional[PositionEncoding] = None,
                rotary_interleaved: bool = False, norm_weights: bool = False, values_from_keys: bool = False,
-               keep_first: int = 0, biases: bool = False, norm_over: str = "head", softcap: float = 0.0, weights: str = "softmax"):
+               keep_first: int = 0, biases: bool = False, norm_over: str = "head", softcap: float = 0.0, weights: str = "softmax",
+               chunk: Optional[int] = None, distance_bias: bool = False, gate_per_head: bool = False):
     super().__init__(name, hidden_size, num_heads, num_kv_heads, dim, scale, norm_eps, rotary, window)
     if values_from_keys and (vdim != dim or value_mix is not None):
       raise ValueError(f"{name}: values that are the keys have the keys' size ({dim}, got vdim={vdim}) and are not mixed")
@@ -63,6 +68,14 @@ class GatedAttentionMixer(AttentionMixer):
       raise ValueError(f"{name}: weights must be 'softmax' or 'sigmoid' (got {weights!r}), and sigmoid weights take no sink")
     if not softcap >= 0:
       raise ValueError(f"{name}: softcap must not be negative, got {softcap!r}")
+    if chunk is not None and (window is not None or chunk < 1):
+      raise ValueError(f"{name}: chunk={chunk} must be positive and goes without a window")
+    if distance_bias and weights != "softmax":
+      raise ValueError(f"{name}: a distance bias goes with a softmax")
+    if gate_per_head and not gated:
+      raise ValueError(f"{name}: gate_per_head without a gate")
+    self.chunk = int(chunk) if chunk is not None else None
+    self.distance_bias, self.gate_per_head = bool(distance_bias), bool(gate_per_head)
     self.softcap = float(softcap)
     self.sigmoid_weights = weights == "sigmoid"
     self.biases = bool(biases)
@@ -83,7 +96,7 @@ class GatedAttentionMixer(AttentionMixer):
     self.value_mix = value_mix
     self.value_mix_key = value_mix_key
     t = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o", "sink": "sink", "mix": "vmix", "q_norm": "q.norm", "k_norm": "k.norm",
-         "q_bias": "q.b", "k_bias": "k.b", "v_bias": "v.b", "score_bias": "pb"}
+         "q_bias": "q.b", "k_bias": "k.b", "v_bias": "v.b", "score_bias": "pb", "r1": "r1", "r2": "r2"}
     t.update(tensors or {})
     self.tensors = t
     H, G = num_heads, num_kv_heads
@@ -91,10 +104,13 @@ class GatedAttentionMixer(AttentionMixer):
     self.k_off = H * dim
     self.v_off = self.k_off if values_from_keys else self.k_off + G * dim
     self.g_off = self.k_off + G * dim + (0 if values_from_keys else G * vdim)
-    self.proj_width = self.g_off + (H * vdim if gated else 0)
+    self.gate_width = 0 if not gated else (H if gate_per_head else H * vdim)
+    self.proj_width = self.g_off + self.gate_width
+    if gate_per_head:      # a gate a head makes an odd number of columns: rows of a size that is read 16 bytes at a time, the rest zero
+      self.proj_width = -(-self.proj_width // 8) * 8
 
   def cache_spec(self) -> Optional[CacheSpec]:
-    return PagedKVSpec(self.num_kv_heads, self.cache_head_dim, self.window, self.keep_first)
+    return PagedKVSpec(self.num_kv_heads, self.cache_head_dim, self.window, self.keep_first, self.chunk)
 
   def param_specs(self) -> Dict[str, ParamSpec]:
     Hd, H, G, D, Dv, n, t = self.hidden_size, self.num_heads, self.num_kv_heads, self.dim, self.vdim, self.name, self.tensors
@@ -102,7 +118,7 @@ class GatedAttentionMixer(AttentionMixer):
     if not self.values_from_keys:
       pieces.append(Piece(f"{n}.{t['v']}", self.v_off, (G * Dv, Hd)))
     if self.gated:
-      pieces.append(Piece(f"{n}.{t['g']}", self.g_off, (H * Dv, Hd)))
+      pieces.append(Piece(f"{n}.{t['g']}", self.g_off, (self.gate_width, Hd)))
     specs = {"qkvg": ParamSpec((self.proj_width, Hd), "matrix", [pieces]),
              "o": ParamSpec((Hd, H * Dv), "matrix", [whole(f"{n}.{t['o']}", (Hd, H * Dv))])}
     if self.norm_weights:
@@ -118,6 +134,8 @@ class GatedAttentionMixer(AttentionMixer):
       specs["sink"] = ParamSpec((H,), "vector", [whole(f"{n}.{t['sink']}", (H,))])
     if self.sigmoid_weights:
       specs["score_bias"] = ParamSpec((H,), "vector", [whole(f"{n}.{t['score_bias']}", (H,))])
+    if self.distance_bias:
+      specs["distance"] = ParamSpec((2 * H,), "vector", [[Piece(f"{n}.{t['r1']}", 0, (H,)), Piece(f"{n}.{t['r2']}", H, (H,))]], init="half_noise")
     if self.value_mix is not None:
       # the layer whose values are the source carries the scalar too (unused), as its file does
       specs["mix"] = ParamSpec((), "vector", [whole(f"{n}.{t['mix']}", ())], init="half_noise")
@@ -129,7 +147,7 @@ class GatedAttentionMixer(AttentionMixer):
     rotary = getattr(self.position, "rotary_dim", None)
     if rotary is not None and rotary > self.dim:
       raise ValueError(f"{self.name}: the rotary encoding covers {rotary} values, more than dim={self.dim}")
-    if dtype == torch.bfloat16 and self.gated:      # the gate's rows are read 16 bytes at a time
+    if dtype == torch.bfloat16 and self.gated and not self.gate_per_head:      # the gate's rows are read 16 bytes at a time
       for what, k in (("width", self.hidden_size), ("heads * vdim", self.num_heads * self.vdim),
                       ("the fused projection's rows", self.proj_width)):
         if k % 8:
@@ -166,7 +184,8 @@ class GatedAttentionMixer(AttentionMixer):
     ops.attention(attn, q_heads, cache.tensor, ctx.block_tables[cache.group], self._batch(ctx), H, G, hdp, self.scale,
                   self.window, sink=self.sink if self.sinks else None, gate=proj if self.gated else None,
                   gate_offset=self.g_off, out_hd=Dv, keep_first=self.keep_first, softcap=self.softcap,
-                  score_bias=self.score_bias if self.sigmoid_weights else None)
+                  score_bias=self.score_bias if self.sigmoid_weights else None, chunk=self.chunk, gate_per_head=self.gate_per_head,
+                  distance=self.distance if self.distance_bias else None)
     out = ctx.ws.buffer(self.out_buffer, (T, self.hidden_size), ctx.dtype)
     ops.linear(out, attn, self.o)
     return out

@@ -15,7 +15,8 @@ values and ``vdim`` value values, a query latent of ``q_rank`` and a key/value l
     denominator if ``sinks``), each giving ``sum_j p_j c_j``, which ``W_uv`` of the head then takes to ``vdim`` values;
   * ``gated``: head h's output is multiplied by ``sigmoid((W_g h)_h)``, one gate a head; then the output projection.
 
-The cache keeps rows of ``kv_rank + rot_dim`` values rounded up to a multiple of 16, zero-filled.  The two per-head
+The cache keeps rows of ``kv_rank + rot_dim`` values rounded up to a multiple of 16, zero-filled (rows of more than 256 values
+take the attention kernel without tensor cores).  The two per-head
 products (``W_uk^T`` on the queries, ``W_uv`` on the outputs) are one batched launch each over the heads of the rows.
 """
 
@@ -85,9 +86,9 @@ class LatentAttentionMixer(AttentionMixer):
       self.uv_heads = params["uv"].view(H, self.vdim, C)
 
   def validate(self, dtype: torch.dtype) -> None:
-    if self.cache_head_dim > 256:
+    if self.cache_head_dim > ops.MAX_HEAD_DIM:
       raise ValueError(f"{self.name}: kv_rank + rot_dim = {self.kv_rank + self.rot_dim} is more than the attention kernels' "
-                       f"largest head size (256)")
+                       f"largest head size ({ops.MAX_HEAD_DIM})")
 
   def takes_residual(self, norm, ctx) -> bool:
     return False

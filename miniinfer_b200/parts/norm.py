@@ -100,20 +100,27 @@ class RMSNorm(Norm):
 
 
 class LayerNorm(Norm):
-  """``(x - mean) / sqrt(var + eps) * weight + bias`` in float32, the variance being the mean of the squared
-  deviations; the residual add (of one or two pending outputs) in front of it, in one kernel.  ``bias_name``: the file
-  tensor of the bias (default ``<name>.bias``; the weight is ``<name>.weight`` or, with ``bare_names``, ``<name>``)."""
+  """``(x - mean) / sqrt(var + eps) * weight (+ bias)`` in float32, the variance being the mean of the squared
+  deviations; the residual add (of one or two pending outputs) in front of it, in one kernel.  ``weight_name``,
+  ``bias_name``: the file tensors (default ``<name>.weight``, ``<name>.bias``).  ``biased`` False: a weight alone."""
 
-  def __init__(self, name: str, dim: int, eps: float, weight_name: Optional[str] = None, bias_name: Optional[str] = None):
+  def __init__(self, name: str, dim: int, eps: float, weight_name: Optional[str] = None, bias_name: Optional[str] = None, biased: bool = True):
     super().__init__(name)
     self.dim = dim
     self.eps = float(eps)
     self.weight_name = weight_name or f"{name}.weight"
     self.bias_name = bias_name or f"{name}.bias"
+    self.biased = bool(biased)
+    self.bias: Optional[torch.Tensor] = None
 
   def param_specs(self) -> Dict[str, ParamSpec]:
-    return {"weight": ParamSpec((self.dim,), "vector", [whole(self.weight_name, (self.dim,))], init="ones_noise"),
-            "bias": ParamSpec((self.dim,), "vector", [whole(self.bias_name, (self.dim,))])}
+    specs = {"weight": ParamSpec((self.dim,), "vector", [whole(self.weight_name, (self.dim,))], init="ones_noise")}
+    if self.biased:
+      specs["bias"] = ParamSpec((self.dim,), "vector", [whole(self.bias_name, (self.dim,))])
+    return specs
+
+  def as_row_norm(self):
+    return "layer", self.weight, self.bias, self.eps
 
   def validate(self, dtype: torch.dtype) -> None:
     if self.dim > 12000:

@@ -140,7 +140,9 @@ def load_weights(spec: ModelSpec, model_dir: str, compute_dtype: torch.dtype, de
   parts_by_id: Dict[int, object] = {}
   for part, local, ps, pieces in plan:
     dt = role_dtype(ps.role, compute_dtype)
-    param = torch.empty(ps.shape, dtype=dt, device=device)
+    # a parameter may be larger than its pieces (rows padded to a size the kernels like): the rest is zero
+    param = (torch.empty if sum(p.shape[0] if p.shape else 1 for p in pieces) == (ps.shape[0] if ps.shape else 1) else torch.zeros)(
+      ps.shape, dtype=dt, device=device)
     for p in pieces:
       src = tensor(fname(p.file_name))
       if ps.role == "int" and src.is_floating_point():

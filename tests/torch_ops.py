@@ -35,7 +35,7 @@ def add_layernorm(out, resid, delta, delta2, weight, bias, eps, rows=None, write
         resid[idx] = x
   mu = x.mean(-1, keepdim=True)
   var = ((x - mu) ** 2).mean(-1, keepdim=True)
-  out.copy_(((x - mu) / torch.sqrt(var + eps) * weight + bias).to(out.dtype))
+  out.copy_(((x - mu) / torch.sqrt(var + eps) * weight + (bias if bias is not None else 0.0)).to(out.dtype))
 
 
 def add_rmsnorm(out, resid, delta, weight, eps, rows=None, write_back=True):
@@ -174,7 +174,7 @@ def _glu(g, u, glu, limit):
 
 
 def routed_experts(out, x, router, correction, gate_up, down, top, workspace, weights="sigmoid_share", glu="silu", limit=0.0,
-                   shared=None, shared_gated=False):
+                   shared=None, shared_gated=False, weight_scale=1.0):
   T, H = x.shape
   E, ff = down.shape[0], down.shape[2]
   z = x.float() @ router.float().t()
@@ -183,14 +183,18 @@ def routed_experts(out, x, router, correction, gate_up, down, top, workspace, we
     w = torch.softmax(torch.gather(z, 1, idx), dim=-1)
   else:
     s = torch.sigmoid(z[:, :E])
-    idx = torch.topk(s + correction, top, dim=-1).indices
+    idx = torch.topk(s + correction if correction is not None else s, top, dim=-1).indices
     w = torch.gather(s, 1, idx)
     w = w / (w.sum(-1, keepdim=True) + 1e-20)
+  w = w * weight_scale
   res = torch.zeros((T, H), dtype=torch.float32, device=x.device)
   for e in range(E):
-    g = x.float() @ gate_up[e, :ff].float().t()
-    u = x.float() @ gate_up[e, ff:].float().t()
-    act = _glu(g, u, glu, limit).to(x.dtype).float()
+    if glu == "relu_squared":
+      act = (torch.relu(x.float() @ gate_up[e].float().t()) ** 2).to(x.dtype).float()
+    else:
+      g = x.float() @ gate_up[e, :ff].float().t()
+      u = x.float() @ gate_up[e, ff:].float().t()
+      act = _glu(g, u, glu, limit).to(x.dtype).float()
     y = act @ down[e].float().t()
     res += (w * (idx == e)).sum(-1, keepdim=True) * y
   if shared is not None:
@@ -264,11 +268,13 @@ def _diagonal(out, a, b, gate, state, ctx, C):
 
 
 def attention(out, qkv, kv_layer, block_table, batch, num_heads, num_kv_heads, head_dim, scale, window,
-              force_generic=False, sink=None, gate=None, gate_offset=0, out_hd=None, keep_first=0, softcap=0.0, score_bias=None):
-  if sink is not None or gate is not None or (out_hd is not None and out_hd != head_dim) or keep_first or softcap or score_bias is not None:
+              force_generic=False, sink=None, gate=None, gate_offset=0, out_hd=None, keep_first=0, softcap=0.0, score_bias=None,
+              chunk=None, gate_per_head=False, distance=None):
+  if (sink is not None or gate is not None or (out_hd is not None and out_hd != head_dim) or keep_first or softcap or score_bias is not None
+      or chunk or distance is not None):
     return _attention_with_options(out, qkv, kv_layer, block_table, batch, num_heads, num_kv_heads, head_dim, scale,
                                    window, sink, gate, gate_offset, out_hd if out_hd is not None else head_dim, keep_first,
-                                   softcap, score_bias)
+                                   softcap, score_bias, chunk, gate_per_head, distance)
   T = qkv.shape[0]
   nh, nkv, hd = num_heads, num_kv_heads, head_dim
   P = kv_layer.shape[3]
@@ -294,7 +300,7 @@ def attention(out, qkv, kv_layer, block_table, batch, num_heads, num_kv_heads, h
 
 
 def _attention_with_options(out, qkv, kv_layer, block_table, batch, nh, nkv, hd, scale, window, sink, gate, gate_offset, ohd,
-                            keep_first=0, softcap=0.0, score_bias=None):
+                            keep_first=0, softcap=0.0, score_bias=None, chunk=None, gate_per_head=False, distance=None):
   T = qkv.shape[0]
   P = kv_layer.shape[3]
   g = nh // nkv
@@ -303,7 +309,7 @@ def _attention_with_options(out, qkv, kv_layer, block_table, batch, nh, nkv, hd,
   res = torch.zeros((T, nh, ohd), dtype=torch.float32, device=qkv.device)
   for t in range(T):
     p = pos[t]
-    lo = max(0, p - window + 1) if window else 0
+    lo = max(0, p - window + 1) if window else (p // chunk * chunk if chunk else 0)
     js = torch.arange(lo, p + 1, device=qkv.device)
     if window and keep_first:
       js = torch.cat((torch.arange(0, min(keep_first, lo), device=qkv.device), js))
@@ -313,6 +319,8 @@ def _attention_with_options(out, qkv, kv_layer, block_table, batch, nh, nkv, hd,
     s = torch.einsum("hd,nhd->hn", q[t], k) * scale
     if softcap:
       s = softcap * torch.tanh(s / softcap)
+    if distance is not None:
+      s = s - distance[:nh, None] * torch.log1p(distance[nh:, None] * (p - js).float())
     if score_bias is not None:
       res[t] = torch.einsum("hn,nhd->hd", torch.sigmoid(s + score_bias[:, None]), v)[:, :ohd]
       continue
@@ -322,7 +330,8 @@ def _attention_with_options(out, qkv, kv_layer, block_table, batch, nh, nkv, hd,
     res[t] = torch.einsum("hn,nhd->hd", pr, v)[:, :ohd]
   res = res.reshape(T, nh * ohd)
   if gate is not None:
-    res = res * torch.sigmoid(gate.float()[:, gate_offset:gate_offset + nh * ohd])
+    g = torch.sigmoid(gate.float()[:, gate_offset:gate_offset + (nh if gate_per_head else nh * ohd)])
+    res = res * (g.repeat_interleave(ohd, dim=1) if gate_per_head else g)
   out.copy_(res.to(out.dtype))
 
 
@@ -466,6 +475,33 @@ def hyper_connection(res, streams, y, mix, out_w, in_w, norm_weight, eps, rows=N
   res.copy_(u.to(res.dtype))
 
 
+def residual_step(out, x, y, mult, x_out, norm=None, rows=None, weights=None, first=None, later=None, n_later=0, keep=None):
+  X = x + mult * y.float() if y is not None else x.clone()
+  if keep is not None:
+    keep.copy_(X)
+  if weights is not None:
+    v = weights[0] * first + weights[n_later + 1] * X
+    for k in range(n_later):
+      v = v + weights[k + 1] * later[k]
+  else:
+    v = X
+  if x_out is not None:
+    x_out.copy_(v)
+  if norm is None:
+    return
+  kind, w, b, eps = norm
+  if rows is not None:
+    v = v[rows.long()]
+  if kind == "layer":
+    v = v - v.mean(-1, keepdim=True)
+  v = v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps) * w
+  out.copy_((v + b if b is not None else v).to(out.dtype))
+
+
+def softcap(x, cap):
+  x.copy_(cap * torch.tanh(x / cap))
+
+
 def relu_squared(out, x):
   out.copy_((torch.relu(x.float()) ** 2).to(out.dtype))
 
@@ -573,5 +609,6 @@ def install(monkeypatch) -> None:
                "attention", "routed_experts", "silu_mul", "sample", "linear_normed", "linear_swiglu_normed", "linear_add",
                "add_rmsnorm_pair", "rms_pair_sum", "linear_batched", "causal_conv", "selective_scan", "gated_delta", "latent_down",
                "latent_query", "linear_attention", "hyper_connection", "relu_squared", "linear_relu_squared", "scaled_pair_sum",
-               "glu_mul", "linear_glu", "linear_parts", "token_shift", "norm_scaled_add", "rglru_recurrence", "mingru_recurrence"):
+               "glu_mul", "linear_glu", "linear_parts", "token_shift", "norm_scaled_add", "rglru_recurrence", "mingru_recurrence",
+               "residual_step", "softcap"):
     monkeypatch.setattr(ops, name, globals()[name])
