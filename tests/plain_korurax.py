@@ -317,3 +317,17 @@ CONFIGS = {
              attention(6, 2, 64, 64, 130, 0.15, moe(32, 6, 2, 1.2)),
              latent(9, 32, 16, 24, 40, 112, 8000.0, 0.2, None)),
 }
+
+
+def peaky_model():
+  """(configuration, weights) under which single keys stand out: chunks of 100 and of 70 tokens, scores spread over tens of
+  units by large scales, distance biases of next to nothing over a chunk, sinks near the largest scores."""
+  cfg = model(200, 64, 1e-5, 0.9, 30.0,
+              attention(4, 2, 64, 64, 100, 0.45, None),
+              latent(2, 32, 16, 32, 32, 48, 10000.0, 0.4, dense(48, 2.0)),
+              attention(2, 1, 32, 48, 70, 0.6, moe(16, 4, 2, 1.0)))
+  W = make_model(cfg, 77)
+  for p in ("l0.mix.", "l2.mix."):
+    W[p + "r1"] = (0.3 * W[p + "r1"]).to(torch.bfloat16).float()
+    W[p + "sink"] = W[p + "sink"] + 6.0
+  return cfg, W

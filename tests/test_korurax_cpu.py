@@ -156,6 +156,42 @@ def test_parts_refuse_options_that_do_not_go_together():
     LMHead("h", 10, 32, softcap=-1.0)
 
 
+def _mistakes():
+  """(what, change of configuration and weights) of mistakes in single mechanisms, planted in the plain implementation."""
+  def chunk(d):
+    return lambda c, W: [x["mixer"]["mask"].__setitem__("size", x["mixer"]["mask"]["size"] + d) for x in c["layers"] if x["type"] == "attention"]
+
+  def scale(suffix, f):
+    return lambda c, W: W.update({k: f(v) for k, v in W.items() if k.endswith(suffix)})
+
+  return [("chunks one longer", chunk(1)), ("chunks one shorter", chunk(-1)), ("no chunks", chunk(100000)),
+          ("no sink", scale(".sink", lambda v: v - 100.0)), ("no distance bias", scale(".r1", lambda v: v * 0)),
+          ("distances half", scale(".r2", lambda v: v * 0.5)), ("gates open", scale("mix.g", lambda v: v * 0)),
+          ("no rotation", lambda c, W: [x["mixer"]["rot"].__setitem__("base", 1e30) for x in c["layers"] if "rot" in x["mixer"]]),
+          ("the last layer alone", scale(".dwa", lambda v: torch.cat((v[:-1] * 0, v[-1:])))),
+          ("no multiplier", lambda c, W: c.__setitem__("residual_mult", 1.0)), ("no cap", lambda c, W: c.__setitem__("logit_softcap", 1e6)),
+          ("another limit", lambda c, W: [x["mlp"].__setitem__("limit", 1e6) for x in c["layers"] if x["mlp"] and x["mlp"]["kind"] == "dense"]),
+          ("another share", lambda c, W: [x["mlp"]["router"].__setitem__("scale", 1.25) for x in c["layers"] if x["mlp"] and x["mlp"]["kind"] == "moe"])]
+
+
+@pytest.mark.parametrize("k", range(13))
+def test_a_mistake_in_one_mechanism_would_show(k):
+  """The weights that the GPU tests run on let every mechanism show: the plain logits with a mistake planted in one of them
+  differ from those without by many times the bound that the engine's float32 logits are held to."""
+  what, change = _mistakes()[k]
+  cfg, W = plain.peaky_model()
+  ids = torch.randint(0, cfg["vocab"], (310,), generator=torch.Generator().manual_seed(6)).tolist()
+  ref = plain.forward(cfg, W, ids)
+  c2, W2 = copy.deepcopy(cfg), dict(W)
+  change(c2, W2)
+  diff = (plain.forward(c2, W2, ids) - ref).abs().max(-1).values
+  bound = 3e-4 * max(1.0, float(ref.pow(2).mean().sqrt()))
+  first = {"chunks one longer": 100, "chunks one shorter": 99, "no chunks": 100}.get(what)
+  if first is not None:      # an edge that is one off moves nothing before it, and the tokens behind it
+    assert float(diff[:69].max()) == 0
+  assert float((diff > 20 * bound).float().mean()) > (0.02 if first else 0.3), (what, float(diff.max()), bound)
+
+
 @pytest.mark.parametrize("tag,page", [("A", 16), ("B", 8), ("C", 64), ("D", 16), ("E", 64)])
 def test_every_cut_gives_the_plain_logits_on_the_host_path(cpu_kernels, tmp_path, tag, page):
   from miniinfer_b200.engine.replay import TraceRunner
