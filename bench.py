@@ -1386,9 +1386,160 @@ def luporax_one(name: str, cfg: dict, size: dict, batch: int, steps: int, warmup
   return out
 
 
+# ---------------------------------------------------------------------------------------------- --compare korurax
+# Sizes for the comparison of the Korurax design with the closest design the engine has, Rikanex (attention with a sink and a
+# gate over a bounded span, a dense first layer and routed experts in the others), at equal size: the sizes of the Rikanex
+# comparison, and for the latent layers those of the Vugudra comparison.  Korurax's layers alternate between latent attention
+# and chunked attention; like Rikanex's its first feed-forward is dense and the others are experts (two matrices each, where
+# Rikanex's have three).  The chunks are such that a decode step at 2048 tokens looks back on about as many keys as Rikanex's
+# window of 1024.
+KORURAX_CHUNK = 1152
+
+
+def korurax_configs(size: dict) -> dict:
+  W, H, G, hd, L = size["width"], size["heads"], size["kv_heads"], size["head"], size["layers"]
+  tag = next(t for t, s in COMPARE_SIZES.items() if s is size)
+  lat = VUGUDRA_SIZES[tag]["latent"]
+  latent = {"type": "latent_attention", "mixer": dict({k: lat[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "q_rank")},
+                                                      scale=(lat["dim"] + lat["rot_dim"]) ** -0.5, rot={"dims": lat["rot_dim"], "base": 10000.0})}
+  chunked = {"type": "attention", "mixer": {"heads": H, "kv_heads": G, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "mask": {"size": KORURAX_CHUNK}}}
+  moe = {"kind": "moe", "expert": {"ff": size["expert_ff"]}, "router": {"experts": size["experts"], "top": size["top"], "scale": 1.5}}
+  dense = {"kind": "dense", "ff": size["ff"], "limit": 7.0}
+  kor = {"architecture": "Korurax", "vocab": COMPARE_VOCAB, "width": W, "norm": {"eps": 1e-6}, "residual_mult": 0.7, "logit_softcap": 30.0,
+         "layers": [dict((latent, chunked)[i % 2], mlp=dense if i == 0 else moe) for i in range(L)]}
+  return {"rikanex": compare_configs(size)["rikanex"], "korurax": kor}
+
+
+def _korurax_groups(times: dict) -> dict:
+  import re
+  g = {"chunked_attention": 0.0, "latent_attention": 0.0, "head_products": 0.0, "experts": 0.0, "routing": 0.0, "dense_products": 0.0,
+       "stream": 0.0, "other": 0.0}
+  for name, us in times.items():
+    if re.search(r"decode_tma_kernel|decode_cluster_kernel|attention_prefill_tc", name):
+      g["chunked_attention"] += us
+    elif re.search(r"decode_split_kernel|decode_merge|attention_prefill_kernel|attention_generic", name):
+      g["latent_attention"] += us      # latent rows of 224 and 256 values
+    elif "gemm_batched" in name:
+      g["head_products"] += us
+    elif "moe_gemm" in name or "moe_stream" in name or re.search(r"gemm_tc_kernel<\w+, \w+, (true|\(bool\)1)[,>]", name):
+      g["experts"] += us
+    elif re.search(r"moe_route|moe_align|moe_combine|moe_gather", name):
+      g["routing"] += us
+    elif "residual_step" in name:
+      g["stream"] += us
+    elif "gemm_skinny" in name or "gemm_tc_kernel" in name or "gemm_stream_tc" in name or \
+        ("anonymous namespace" not in name and re.search(r"nvjet|cutlass|cublas|gemm|gemv|xmma", name, re.I)):
+      g["dense_products"] += us
+    elif not name.startswith("Memcpy") and not name.startswith("Memset"):
+      g["other"] += us
+  return {k: max(v, 1e-9) for k, v in g.items()}
+
+
+def _step_kernel_times(engine, batch: int) -> tuple:
+  """(kernel times of a decode step, of a 2048-token prefill step, row tiles of the last routed layer that an expert owns)."""
+  import torch
+  from miniinfer_b200.engine import StepItem
+  from miniinfer_b200.sampling import Sampler, SamplingParams
+  rids = fill_context(engine, batch, CONTEXT, seed=1000 + batch)
+  params = [SamplingParams(temperature=0.6, max_tokens=GENERATED, ignore_eos=True)] * batch
+  tokens_dev = torch.zeros(max(batch, 1), dtype=torch.int32, device="cuda:0")
+
+  def decode(i):
+    engine.runner.step_and_sample([StepItem(r, [1], (0,)) for r in rids], Sampler.pack(params, list(range(batch)), [i] * batch),
+                                  Sampler.sample, tokens_dev, sampling_pad=Sampler.PAD_ROWS)
+
+  for i in range(4):
+    decode(i)
+  torch.cuda.synchronize()
+  dtimes = _kernel_times(lambda i: decode(10 + i), 4)
+  touched = 0.0
+  for gph in engine.runner._graphs.values():
+    buf = gph.ws._bufs.get(("moe_tile_expert", torch.int32))
+    if buf is not None:
+      touched = float((buf >= 0).sum().item())
+  for r in rids:
+    engine.cache.release_request(r)
+  g = torch.Generator().manual_seed(7)
+
+  def whole(i):
+    engine.cache.admit(f"rates{i}")
+    engine.runner.step([StepItem(f"rates{i}", torch.randint(0, COMPARE_VOCAB, (PREFILL_TOKENS,), generator=g).tolist(), (PREFILL_TOKENS - 1,))])
+    engine.cache.release_request(f"rates{i}")
+
+  for i in range(2):
+    whole(i)
+  torch.cuda.synchronize()
+  return dtimes, _kernel_times(lambda i: whole(10 + i), 2), touched
+
+
+def korurax_one(name: str, cfg: dict, size: dict, batch: int, steps: int, warmup: int, pk: dict, kernels: bool) -> dict:
+  """Prefill and decode of one model of the comparison; with ``kernels`` the device time of its kinds of kernels and the
+  rates they reach against the measured peaks (run with dependent launch off, see main)."""
+  if name == "rikanex":
+    return compare_one(name, cfg, size, batch, steps, warmup, pk, kernels)
+  import torch
+  W, H, G, hd, L, T = size["width"], size["heads"], size["kv_heads"], size["head"], size["layers"], PREFILL_TOKENS
+  with tempfile.TemporaryDirectory() as d:
+    with open(os.path.join(d, "config.json"), "w") as f:
+      json.dump(cfg, f)
+    engine = build_engine(d, batch)
+    if not kernels:
+      dec = time_decode(engine, batch, steps, warmup)
+      pre = time_prefill(engine)
+      out = {"decode_tok_s": round(dec["tok_s"], 1), "decode_ms": round(dec["ms"], 4), "launches_per_decode_step": int(dec["launches_per_step"]),
+             "prefill_tok_s": round(T / (pre["ms"] * 1e-3), 1), "prefill_ms": round(pre["ms"], 3)}
+    else:
+      dtimes, ptimes, touched = _step_kernel_times(engine, batch)
+      dk, pt = _korurax_groups(dtimes), _korurax_groups(ptimes)
+      lat = cfg["layers"][0]["mixer"]
+      lH, D, R, Dv, C, Q = (lat[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "q_rank"))
+      n_lat, n_att, n_moe = (L + 1) // 2, L // 2, L - 1
+      E, F, top = size["experts"], size["expert_ff"], size["top"]
+      keys = CONTEXT % KORURAX_CHUNK
+      row = -(-(C + R) // 16) * 16
+      att_flops = n_att * 4.0 * H * hd * sum(t % KORURAX_CHUNK + 1 for t in range(T))
+      lat_flops = n_lat * 2.0 * lH * (C + R + C) * sum(t + 1 for t in range(T))
+      moe_flops, moe_bytes = n_moe * T * top * 2 * 2.0 * F * W, n_moe * touched * 2 * F * W * 2
+      proj_w = n_att * ((2 * H + 2 * G) * hd * W + H * W) + n_lat * ((Q + C + R) * W + lH * (D + R) * Q + lH * Dv * W) + 3 * size["ff"] * W
+      head_w = n_lat * lH * (D + Dv) * C
+      # a stream step reads the float32 row and the sublayer's output and writes row and normed rounding; at a layer's end it
+      # also reads the embedding's row and every earlier result and writes this layer's
+      stream = sum((4 + 2 + 4 + 2) * W + (4 + 2 + 4 + 2) * W + 4 * W * (i + 1) + (4 * W if i + 1 < L else 0) for i in range(L))
+
+      def rate(us, amount, peak, unit):      # amount in FLOP or bytes
+        v = amount / us / (1e6 if unit == "TFLOP/s" else 1e3)
+        return {"us": round(us, 1), unit: round(v, 1), "frac": round(v / peak, 4)}
+
+      tf, gb = pk["bf16_tflops"], pk["hbm_gbs"]
+      out = {"prefill_chunked_attention": rate(pt["chunked_attention"], att_flops, tf, "TFLOP/s"),
+             "decode_chunked_attention": rate(dk["chunked_attention"], batch * keys * n_att * 2 * G * hd * 2, gb, "GB/s"),
+             "prefill_latent_attention": rate(pt["latent_attention"], lat_flops, tf, "TFLOP/s"),
+             "decode_latent_attention": rate(dk["latent_attention"], batch * CONTEXT * n_lat * 2 * row * 2, gb, "GB/s"),
+             "prefill_head_products": rate(pt["head_products"], 2.0 * T * head_w, tf, "TFLOP/s"),
+             "decode_head_products": rate(dk["head_products"], 2.0 * head_w, gb, "GB/s"),
+             "prefill_experts": rate(pt["experts"], moe_flops, tf, "TFLOP/s"),
+             "decode_experts": dict(rate(dk["experts"], moe_bytes, gb, "GB/s"), experts_read_per_layer=round(touched, 1)),
+             "routing_us": {"prefill": round(pt["routing"], 1), "decode": round(dk["routing"], 1)},
+             "prefill_dense_products": rate(pt["dense_products"], 2.0 * T * proj_w, tf, "TFLOP/s"),
+             "decode_dense_products": rate(dk["dense_products"], 2.0 * (proj_w + COMPARE_VOCAB * W), gb, "GB/s"),
+             "prefill_stream": rate(pt["stream"], T * stream, gb, "GB/s"), "decode_stream_us": round(dk["stream"], 1),
+             "other_us": {"prefill": round(pt["other"], 1), "decode": round(dk["other"], 1)}}
+
+      def top_of(times):
+        rows = sorted(((us, n) for n, us in times.items() if not n.startswith("Mem")), reverse=True)[:14]
+        return [[round(us, 1), n.replace("(anonymous namespace)::", "")[:70]] for us, n in rows]
+
+      out["top_kernels_us"] = {"prefill": top_of(ptimes), "decode": top_of(dtimes)}
+    engine.stop()
+    del engine
+    gc.collect()
+    torch.cuda.empty_cache()
+  return out
+
+
 def compare_designs(args) -> int:
   """``--compare rikanex`` / ``--compare vugudra``: the design beside the Qwen3 dense decoder at equal sizes (random weights);
-  ``--compare famupel``: the design beside Vugudra, ``--compare luporax``: the design beside Rikanex, each the closest of
+  ``--compare famupel``: the design beside Vugudra, ``--compare luporax`` and ``--compare korurax``: the design beside Rikanex, each the closest of
   the engine's designs, at equal sizes: prefill of
   one 2048-token prompt and decode steps at ``--batch`` requests with ``--context``-token contexts, and, from a process of
   its own with dependent launch off, what the kinds of kernels of both reach against the measured peaks."""
@@ -1401,8 +1552,9 @@ def compare_designs(args) -> int:
   design = args.compare
   sizes_of, configs_of, one = {"rikanex": (COMPARE_SIZES, compare_configs, compare_one), "vugudra": (VUGUDRA_SIZES, vugudra_configs, vugudra_one),
                                "famupel": (FAMUPEL_SIZES, famupel_configs, famupel_one),
-                               "luporax": (COMPARE_SIZES, luporax_configs, luporax_one)}[design]
-  beside = {"famupel": "vugudra", "luporax": "rikanex"}.get(design, "qwen3")
+                               "luporax": (COMPARE_SIZES, luporax_configs, luporax_one),
+                               "korurax": (COMPARE_SIZES, korurax_configs, korurax_one)}[design]
+  beside = {"famupel": "vugudra", "luporax": "rikanex", "korurax": "rikanex"}.get(design, "qwen3")
   result = {"compare": f"{design} beside {beside} at equal sizes", "batch": args.batch, "context": CONTEXT, "window": COMPARE_WINDOW,
             "vocab": COMPARE_VOCAB, "prefill_tokens": PREFILL_TOKENS, "steps": args.steps, "warmup": warmup, "dtype": "bf16",
             "data": "synthetic: random weights, uniform random token ids", "peaks": pk["source"], "sizes": {}}
@@ -1441,8 +1593,8 @@ def main() -> int:
   ap.add_argument("--steps", type=int, default=128)
   ap.add_argument("--warmup", type=int, default=8)
   ap.add_argument("--impl", default="ours", choices=["ours", "reference", "reference-child", "kernels-child", "compare-child"])
-  ap.add_argument("--compare", default=None, choices=["rikanex", "vugudra", "famupel", "luporax"],
-                  help="time the Rikanex or the Vugudra design beside the Qwen3 dense decoder, the Famupel design beside Vugudra, or the Luporax design beside Rikanex, at equal sizes (--sizes), print one JSON line and exit")
+  ap.add_argument("--compare", default=None, choices=["rikanex", "vugudra", "famupel", "luporax", "korurax"],
+                  help="time the Rikanex or the Vugudra design beside the Qwen3 dense decoder, the Famupel design beside Vugudra, or the Luporax or the Korurax design beside Rikanex, at equal sizes (--sizes), print one JSON line and exit")
   ap.add_argument("--sizes", default="s,m,l", help="with --compare: which of the sizes s, m, l (commas between them)")
   ap.add_argument("--batch", type=int, default=8)
   ap.add_argument("--shape", default="0.6b", choices=sorted(SHAPES), help="layer sizes: the default, or another Qwen3 model's")
