@@ -1420,7 +1420,7 @@ def _korurax_groups(times: dict) -> dict:
     elif re.search(r"decode_split_kernel|decode_merge|attention_prefill_kernel|attention_generic", name):
       g["latent_attention"] += us      # latent rows of 224 and 256 values
     elif "gemm_batched" in name:
-      g["head_products"] += us
+      g["head_products"] += us      # (the library's products of a prefill step are among the dense products)
     elif "moe_gemm" in name or "moe_stream" in name or re.search(r"gemm_tc_kernel<\w+, \w+, (true|\(bool\)1)[,>]", name):
       g["experts"] += us
     elif re.search(r"moe_route|moe_align|moe_combine|moe_gather", name):
@@ -1515,12 +1515,11 @@ def korurax_one(name: str, cfg: dict, size: dict, batch: int, steps: int, warmup
              "decode_chunked_attention": rate(dk["chunked_attention"], batch * keys * n_att * 2 * G * hd * 2, gb, "GB/s"),
              "prefill_latent_attention": rate(pt["latent_attention"], lat_flops, tf, "TFLOP/s"),
              "decode_latent_attention": rate(dk["latent_attention"], batch * CONTEXT * n_lat * 2 * row * 2, gb, "GB/s"),
-             "prefill_head_products": rate(pt["head_products"], 2.0 * T * head_w, tf, "TFLOP/s"),
              "decode_head_products": rate(dk["head_products"], 2.0 * head_w, gb, "GB/s"),
              "prefill_experts": rate(pt["experts"], moe_flops, tf, "TFLOP/s"),
              "decode_experts": dict(rate(dk["experts"], moe_bytes, gb, "GB/s"), experts_read_per_layer=round(touched, 1)),
              "routing_us": {"prefill": round(pt["routing"], 1), "decode": round(dk["routing"], 1)},
-             "prefill_dense_products": rate(pt["dense_products"], 2.0 * T * proj_w, tf, "TFLOP/s"),
+             "prefill_dense_products": rate(pt["dense_products"] + pt["head_products"], 2.0 * T * (proj_w + head_w), tf, "TFLOP/s"),
              "decode_dense_products": rate(dk["dense_products"], 2.0 * (proj_w + COMPARE_VOCAB * W), gb, "GB/s"),
              "prefill_stream": rate(pt["stream"], T * stream, gb, "GB/s"), "decode_stream_us": round(dk["stream"], 1),
              "other_us": {"prefill": round(pt["other"], 1), "decode": round(dk["other"], 1)}}

@@ -2,11 +2,12 @@
 // number of new tokens at any offset) against all keys of their request that the mask allows.
 //
 // A block of four warps owns 64 query rows of one request and one query head (a "tile" of the
-// step's work list); each warp owns 16 rows.  It walks the keys in blocks of 64: K and V rows are
+// step's work list); each warp owns 16 rows.  Head sizes above 128 leave room for one block an SM only: there a block
+// has eight warps and takes two neighbouring query heads of a kv head, which share the keys and values it gathers.  It walks the keys in blocks of 64: K and V rows are
 // gathered page by page into shared memory with cp.async (two stages: the next block loads while
 // this one is multiplied), S = Q K^T and O += P V run as mma.m16n8k16 (bf16 in, fp32 accumulate),
 // softmax is the online form in float32 with exp2 and the scale folded in, P is rounded to bf16
-// for the second product.  Causal and window masks are applied by absolute position, so a portion
+// for the second product.  Causal, window and chunk masks are applied by absolute position, so a portion
 // that starts in the middle of a prompt sees the cached keys before it.
 //
 // Shared-memory rows are padded by 16 bytes; with head sizes that are multiples of 16 the row
@@ -40,7 +41,7 @@ namespace {
 constexpr int HD = MI_HEAD_DIM;
 constexpr int BQ = 64;            // query rows of a tile
 constexpr int BK = 64;            // keys of a block
-constexpr int WARPS = 4;
+constexpr int WARPS = 4;          // of a query head
 constexpr int LDS = HD + 8;       // shared-memory row stride in elements
 constexpr int CHUNKS = HD / 8;    // 16-byte chunks of a row
 constexpr int KSTEPS = HD / 16;   // k16 steps of Q K^T
@@ -100,9 +101,10 @@ struct PrefillArgs {
 };
 
 // Gathers keys kb*BK .. kb*BK+BK of one kv head (K and V) into a stage; rows past `last_key` are zeros.
+template <int HEADS>
 __device__ __forceinline__ void load_kv_block(__nv_bfloat16* ks, __nv_bfloat16* vs, const PrefillArgs& a, const int* bt,
                                               size_t page_elems, size_t head_off, size_t v_off, int kb, int last_key) {
-  for (int idx = threadIdx.x; idx < BK * CHUNKS; idx += WARPS * 32) {
+  for (int idx = threadIdx.x; idx < BK * CHUNKS; idx += HEADS * WARPS * 32) {
     const int r = idx / CHUNKS, c = idx % CHUNKS;
     const int j = kb * BK + r;
     const bool valid = j <= last_key;
@@ -116,20 +118,21 @@ __device__ __forceinline__ void load_kv_block(__nv_bfloat16* ks, __nv_bfloat16* 
   }
 }
 
-// SHAPED: the form for shaped scores, compiled apart so that the plain softmax carries none of it.
-template <bool SHAPED>
-__global__ void __launch_bounds__(WARPS * 32)
+// SHAPED: the form for shaped scores, compiled apart so that the plain softmax carries none of it.  HEADS: query heads of a block.
+template <bool SHAPED, int HEADS>
+__global__ void __launch_bounds__(HEADS * WARPS * 32)
 attention_prefill_kernel(PrefillArgs a) {
   mi::grid_dependency_sync();
   extern __shared__ __align__(16) unsigned char smem_raw[];
-  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(smem_raw);   // [BQ][LDS]
-  __nv_bfloat16* kbuf = qs + BQ * LDS;                              // [2][BK][LDS]
+  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(smem_raw);   // [HEADS][BQ][LDS]
+  __nv_bfloat16* kbuf = qs + HEADS * BQ * LDS;                              // [2][BK][LDS]
   __nv_bfloat16* vbuf = kbuf + 2 * BK * LDS;                        // [2][BK][LDS]
 
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int lane = threadIdx.x & 31, warp = (threadIdx.x >> 5) % WARPS, sub = (threadIdx.x >> 5) / WARPS;   // warp of its head, head of the block
   const int g = lane >> 2, t = lane & 3;
-  const int item = a.tiles[2 * blockIdx.x], off = a.tiles[2 * blockIdx.x + 1];
-  const int head = blockIdx.y;
+  const int tile = (int)(gridDim.x - 1 - blockIdx.x);          // an item's last tiles see the most keys: they start first
+  const int item = a.tiles[2 * tile], off = a.tiles[2 * tile + 1];
+  const int head = blockIdx.y * HEADS + sub;
   const int kvh = head / (a.nh / a.nkv);
   const int n_new = a.q_len[item];
   const int rows = min(BQ, n_new - off);
@@ -147,13 +150,13 @@ attention_prefill_kernel(PrefillArgs a) {
   const size_t v_off = (size_t)a.nkv * a.page_size * HD;
 
   // Q tile -> shared memory (rows past the portion are zeros), with the first K/V block behind it
-  for (int idx = threadIdx.x; idx < BQ * CHUNKS; idx += WARPS * 32) {
-    const int r = idx / CHUNKS, c = idx % CHUNKS;
+  for (int idx = threadIdx.x; idx < HEADS * BQ * CHUNKS; idx += HEADS * WARPS * 32) {
+    const int hr = idx / CHUNKS, c = idx % CHUNKS, r = hr % BQ;
     const bool valid = r < rows;
-    const __nv_bfloat16* src = valid ? a.q_base + (size_t)(row0 + r) * a.q_stride + (size_t)head * HD + c * 8 : a.q_base;
-    cp_async16(qs + r * LDS + c * 8, src, valid);
+    const __nv_bfloat16* src = valid ? a.q_base + (size_t)(row0 + r) * a.q_stride + (size_t)(blockIdx.y * HEADS + hr / BQ) * HD + c * 8 : a.q_base;
+    cp_async16(qs + hr * LDS + c * 8, src, valid);
   }
-  load_kv_block(kbuf, vbuf, a, bt, page_elems, head_off, v_off, n_first > 0 ? 0 : kb_begin, p_last);
+  load_kv_block<HEADS>(kbuf, vbuf, a, bt, page_elems, head_off, v_off, n_first > 0 ? 0 : kb_begin, p_last);
   cp_async_commit();
 
   uint32_t qf[Q_IN_REGS ? KSTEPS : 1][4];
@@ -164,6 +167,7 @@ attention_prefill_kernel(PrefillArgs a) {
     for (int c = 0; c < 4; ++c) o[i][c] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
   const int pr[2] = {p0 + warp * 16 + g, p0 + warp * 16 + g + 8};    // positions of this thread's two rows
+  const int lo_last = mi::first_visible(p_last, a.window), kept = a.window > 0 ? a.keep_first : 0;
   const bool row_ok[2] = {warp * 16 + g < rows, warp * 16 + g + 8 < rows};
   const bool shaped = SHAPED, sigmoid = SHAPED && a.score_bias != nullptr;
   const float head_bias = sigmoid ? a.score_bias[head] : 0.f;
@@ -173,7 +177,7 @@ attention_prefill_kernel(PrefillArgs a) {
 
   // ldmatrix lane addressing: lane l gives the row address of 8x8 matrix l/8, row l%8
   const int lm = lane >> 3, lr = lane & 7;
-  const __nv_bfloat16* q_lane = qs + (warp * 16 + (lm & 1) * 8 + lr) * LDS + (lm >> 1) * 8;
+  const __nv_bfloat16* q_lane = qs + (sub * BQ + warp * 16 + (lm & 1) * 8 + lr) * LDS + (lm >> 1) * 8;
 
   for (int bi = 0; bi < n_blocks; ++bi) {
     const int kb = bi < n_first ? bi : kb_begin + (bi - n_first);
@@ -182,7 +186,7 @@ attention_prefill_kernel(PrefillArgs a) {
     __nv_bfloat16* ks = kbuf + stage * BK * LDS;
     __nv_bfloat16* vs = vbuf + stage * BK * LDS;
     if (bi + 1 < n_blocks) {
-      load_kv_block(kbuf + (stage ^ 1) * BK * LDS, vbuf + (stage ^ 1) * BK * LDS, a, bt, page_elems, head_off, v_off, kb_next, p_last);
+      load_kv_block<HEADS>(kbuf + (stage ^ 1) * BK * LDS, vbuf + (stage ^ 1) * BK * LDS, a, bt, page_elems, head_off, v_off, kb_next, p_last);
       cp_async_commit();
       cp_async_wait<1>();
     } else {
@@ -219,20 +223,32 @@ attention_prefill_kernel(PrefillArgs a) {
       }
     }
 
-    // mask by absolute position, online softmax in float32 (base 2, scale folded in)
+    // Mask by absolute position (only in blocks that the mask of some row touches), online softmax in float32 (base 2, scale
+    // folded in).
+    const bool inside = rows == BQ && kb * BK + BK - 1 <= p0 && kb * BK >= lo_last;
     float mx[2] = {-INFINITY, -INFINITY};
+    if (SHAPED || !inside) {
 #pragma unroll
-    for (int i = 0; i < NT_S; ++i)
+      for (int i = 0; i < NT_S; ++i)
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        const int j = kb * BK + i * 8 + 2 * t + (c & 1);
-        const int h = c >> 1;
-        const bool see = row_ok[h] && j <= pr[h] && (j >= lo_row[h] || (a.window > 0 && j < a.keep_first));
-        float v = see ? (shaped ? mi::shaped_logit2(s[i][c], a.scale, a.softcap, sigmoid, head_bias) : s[i][c] * a.scale_log2) : -INFINITY;
-        if (distance && see) v -= mi::distance_logit2(r1, r2, pr[h] - j);
-        s[i][c] = v;
-        mx[h] = fmaxf(mx[h], v);
-      }
+        for (int c = 0; c < 4; ++c) {
+          const int j = kb * BK + i * 8 + 2 * t + (c & 1);
+          const int h = c >> 1;
+          const bool see = row_ok[h] && j <= pr[h] && (j >= lo_row[h] || j < kept);
+          float v = see ? (shaped ? mi::shaped_logit2(s[i][c], a.scale, a.softcap, sigmoid, head_bias) : s[i][c] * a.scale_log2) : -INFINITY;
+          if (distance && see) v -= mi::distance_logit2(r1, r2, pr[h] - j);
+          s[i][c] = v;
+          mx[h] = fmaxf(mx[h], v);
+        }
+    } else {
+#pragma unroll
+      for (int i = 0; i < NT_S; ++i)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          s[i][c] *= a.scale_log2;
+          mx[c >> 1] = fmaxf(mx[c >> 1], s[i][c]);
+        }
+    }
     float alpha[2], m_use[2];
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
@@ -316,6 +332,19 @@ attention_prefill_kernel(PrefillArgs a) {
   }
 }
 
+template <bool SHAPED, int HEADS>
+int launch_prefill(const PrefillArgs& a, int n_tiles, cudaStream_t stream) {
+  constexpr size_t smem = (size_t)(HEADS * BQ + 4 * BK) * LDS * sizeof(__nv_bfloat16);
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel<SHAPED, HEADS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return mi_fail("attention_prefill: cannot get %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
+    configured = true;
+  }
+  mi::launch(attention_prefill_kernel<SHAPED, HEADS>, dim3(n_tiles, a.nh / HEADS), dim3(HEADS * WARPS * 32), smem, stream, a);
+  return 0;
+}
+
 }  // namespace
 
 MI_API int mi_attention_head_dim() { return HD; }
@@ -347,16 +376,12 @@ MI_API int mi_attention_prefill_bf16(void* out, const void* q_base, int q_stride
   a.scale_log2 = scale * 1.4426950408889634f;
   a.sink = sink; a.gate = (const __nv_bfloat16*)gate; a.gate_stride = gate_stride; a.out_hd = out_hd;
   a.scale = scale; a.softcap = softcap; a.score_bias = score_bias; a.gate_per_head = gate_per_head; a.distance = distance;
-  const size_t smem = (size_t)(BQ + 4 * BK) * LDS * sizeof(__nv_bfloat16);
-  static bool configured = false;
-  if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(attention_prefill_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) return mi_fail("attention_prefill: cannot get %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
-    configured = true;
-  }
-  if (softcap > 0.f || score_bias != nullptr || distance != nullptr) mi::launch(attention_prefill_kernel<true>, dim3(dim3(n_tiles, nh)), dim3(WARPS * 32), smem, stream, a);
-  else mi::launch(attention_prefill_kernel<false>, dim3(dim3(n_tiles, nh)), dim3(WARPS * 32), smem, stream, a);
+  const bool is_shaped = softcap > 0.f || score_bias != nullptr || distance != nullptr;
+  constexpr int WIDE = HD > 128 ? 2 : 1;      // query heads of a block where the head size leaves room for one block an SM
+  int rc;
+  if (WIDE == 2 && (nh / nkv) % 2 == 0) rc = is_shaped ? launch_prefill<true, WIDE>(a, n_tiles, stream) : launch_prefill<false, WIDE>(a, n_tiles, stream);
+  else rc = is_shaped ? launch_prefill<true, 1>(a, n_tiles, stream) : launch_prefill<false, 1>(a, n_tiles, stream);
+  if (rc) return rc;
   MI_LAUNCH_OK("attention_prefill");
   return 0;
 }

@@ -144,6 +144,15 @@ constexpr int OUT_ROW_BYTES = HD;                       // a softmax thread's ha
 constexpr size_t SMEM_BYTES = 1024 + Q_BYTES + KV_RING_BYTES + 256 + (2 * STREAMS * TPR + 2 * STREAMS * (TPR + 1)) * BM * sizeof(float) +
                               (size_t)SOFTMAX_WARPS * 32 * OUT_ROW_BYTES;
 
+// Distance biases: r1 log2(1 + r2 d) for every distance of a work's rows and keys, per head, worked out once a work - read
+// from shared memory it costs the softmax threads no second logarithm-sized operation a score beside the exponential (the
+// special-function unit takes one value in eight cycles of a warp).  TABLE_PAD entries stand for the keys ahead of a row.
+// Works whose keys reach back further than the table work the logarithm out score by score.
+constexpr size_t TABLE_ROOM = (227 * 1024 - SMEM_BYTES) / sizeof(float);
+constexpr int TABLE = TABLE_ROOM < 16384 ? (int)TABLE_ROOM / 2 * 2 : 16384;      // entries, of one head or of two
+constexpr int TABLE_PAD = 2 * BN;
+template <int SCORES> constexpr size_t smem_bytes_of() { return SMEM_BYTES + (SCORES == 3 ? TABLE * sizeof(float) : 0); }
+
 // two bf16 outputs times the sigmoid of two bf16 gate logits
 __device__ __forceinline__ uint32_t gate_pair(uint32_t o2, uint32_t g2) {
   const float2 o = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&o2));
@@ -692,6 +701,20 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
       const bool row_valid = tok < rows_tok;
       const int pos = row_valid ? start + o + tok : p_last;
       const int lo_r = mi::first_visible(pos, a.window);
+      // The table of this work's heads: the softmax warps have all met since the last one was read (at the end of a work).
+      const float* to_row = nullptr;
+      if constexpr (distance) {
+        float* table = reinterpret_cast<float*>(out_s + SOFTMAX_WARPS * 32 * OUT_ROW_BYTES);
+        const int room = TABLE / a.hpt, need = p_last - t_begin * BN + 1 + TABLE_PAD;
+        if (wk.n_first == 0 && need <= room) {
+          for (int idx = (int)threadIdx.x; idx < need * a.hpt; idx += SOFTMAX_WARPS * 32) {
+            const int hh = idx >= need ? 1 : 0, d = idx - hh * need;
+            table[hh * room + d] = mi::distance_logit2(a.distance[wk.head0 + hh], a.distance[a.nh + wk.head0 + hh], max(d - TABLE_PAD, 0));
+          }
+          asm volatile("bar.sync 8, %0;" ::"n"(SOFTMAX_WARPS * 32) : "memory");
+          to_row = table + (a.hpt == 2 ? (r >> 6) * room : 0) + pos + TABLE_PAD;
+        }
+      }
       float m_run = -INFINITY, l_run = 0.f;
       const int n_mine = (n - st + 1) / 2;                 // tiles of this stream
       const float head_bias = sigmoid ? a.score_bias[head] : 0.f;
@@ -716,7 +739,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
         } else if (distance) {
           // keys behind the query only: what lies ahead (a logarithm of nothing) is hidden below
           const float at0 = fmaf(r2, (float)(pos - key0), 1.f);      // 1 + r2 d of the tile's first key
-          if (a.softcap > 0.f) {
+          if (to_row != nullptr && !(a.softcap > 0.f)) {
+            const float* to = to_row - key0;                          // a key's entry lies at its distance: one further back, one entry further up
+#pragma unroll
+            for (int e = 0; e < BN; ++e) v[e] = fmaf(v[e], a.scale_log2, -to[-e]);
+          } else if (a.softcap > 0.f) {
 #pragma unroll
             for (int e = 0; e < BN; ++e)
               v[e] = fmaf(-r1, mi::lg2_fast(fmaf(-r2, (float)e, at0)), mi::shaped_logit2(v[e], a.scale, a.softcap, false, 0.f));
@@ -933,13 +960,13 @@ int launch_prefill_tc(const CUtensorMap& qm, const CUtensorMap& km, const Args& 
   auto kernel = attention_prefill_tc_kernel<CTAS, SCORES>;
   static bool configured = false;
   if (!configured) {
-    cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);
-    if (err != cudaSuccess) return mi_fail("attention_prefill_tc: cannot get %zu bytes of shared memory: %s", SMEM_BYTES, cudaGetErrorString(err));
+    cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_bytes_of<SCORES>());
+    if (err != cudaSuccess) return mi_fail("attention_prefill_tc: cannot get %zu bytes of shared memory: %s", smem_bytes_of<SCORES>(), cudaGetErrorString(err));
     configured = true;
   }
   cudaLaunchConfig_t cfg = {};
   cfg.blockDim = dim3(THREADS);
-  cfg.dynamicSmemBytes = SMEM_BYTES;
+  cfg.dynamicSmemBytes = smem_bytes_of<SCORES>();
   cfg.stream = stream;
   cudaLaunchAttribute attr[2];
   int n_attr = 0;

@@ -498,7 +498,8 @@ def linear_batched(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, bias: Op
                    row_gate: Optional[torch.Tensor] = None) -> None:
   """out[:, b, :] = x[:, b, :] @ w[b]^T for ``x [M, batch, K]``, ``w [batch, N, K]``, ``out [M, batch, N]`` - views whose
   strides may be anything as long as the last axis is contiguous (the heads of a token's row, a column range of a
-  row); float32 sums, k ascending.  ``bias [N]`` float32 is added, ``softplus`` applied, and with ``row_gate [M, >= batch]``
+  row); float32 sums, k ascending.  bfloat16 with more than 16 rows and nothing behind the product: one strided batched library product.
+  ``bias [N]`` float32 is added, ``softplus`` applied, and with ``row_gate [M, >= batch]``
   (one logit per row and batch) the result is multiplied with its sigmoid."""
   lib = common_lib()
   M, B, K = x.shape
@@ -516,6 +517,18 @@ def linear_batched(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, bias: Op
       raise KernelError("linear_batched: the row gate must hold a logit per row and batch, in the operands' dtype")
     gate_stride = row_gate.stride(0)
   few = M <= 16 and x.dtype == torch.bfloat16
+  aligned = K % 8 == 0 and all(t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0 and t.stride(1) % 8 == 0 for t in (x, w, out))
+  if (x.dtype == torch.bfloat16 and not few and out.dtype == torch.bfloat16 and bias is None and row_gate is None and not softplus
+      and B > 1 and w.stride(1) == K and aligned):
+    # many rows and nothing behind the product: the library's, all parts in one call (torch's while a graph is recorded)
+    if not _capturing:
+      _check(lib, lib.mi_gemm_cublas_bf16_batched(
+        ctypes.c_void_p(out.data_ptr()), _dt(out), ctypes.c_void_p(x.data_ptr()), ctypes.c_void_p(w.data_ptr()), M, N, K, int(x.stride(0)),
+        ctypes.c_longlong(x.stride(1)), ctypes.c_longlong(w.stride(0)), int(out.stride(0)), ctypes.c_longlong(out.stride(1)), B, _stream()),
+        kernels=0)
+    else:
+      torch.bmm(x.transpose(0, 1), w.transpose(1, 2), out=out.transpose(0, 1))
+    return
   _check(lib, (lib.mi_gemm_batched_few_rows if few else lib.mi_gemm_batched)(
     ctypes.c_void_p(out.data_ptr()), _dt(out), ctypes.c_void_p(x.data_ptr()), ctypes.c_void_p(w.data_ptr()), _dt(x), B, M, N, K,
     int(x.stride(0)), ctypes.c_longlong(x.stride(1)), int(w.stride(1)), ctypes.c_longlong(w.stride(0)),
@@ -537,7 +550,7 @@ def linear_parts(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor) -> None:
     if not _capturing:
       lib = common_lib()
       _check(lib, lib.mi_gemm_cublas_bf16_batched(_ptr(out), _dt(out), _ptr(x), _ptr(w), M, N, K, B * K, ctypes.c_longlong(K),
-                                                  ctypes.c_longlong(N * K), ctypes.c_longlong(M * N), B, _stream()), kernels=0)
+                                                  ctypes.c_longlong(N * K), N, ctypes.c_longlong(M * N), B, _stream()), kernels=0)
       return
     # while a graph is recorded: torch's products, a part at a time (float32 results where this torch build writes them)
     if out.dtype == torch.bfloat16 or _mm_f32_out_works(out.device):

@@ -194,6 +194,24 @@ def test_single_keys_that_stand_out_in_prompts_and_in_decoding(tmp_path, dtype, 
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("tag", ["C", "E"])
+def test_steps_of_one_shape_that_are_replayed(korurax_dirs, dtype, tag):
+  """Five prompts of one length whole, one after the other, then their tails in portions of one size: from the second step of
+  a shape on it is recorded and replayed, with other pages and other tokens each time."""
+  d = korurax_dirs(tag)
+  reqs = rc.make_requests(plain.CONFIGS[tag]["vocab"], (150,) * 5, seed=31)
+  ref = reference(d, reqs)
+  trace = []
+  for rid, ids in reqs.items():
+    for lo, hi in ((0, 100), (100, 125), (125, 150)):
+      trace.append({"step": len(trace), "entries": [{"id": rid, "tokens": ids[lo:hi], "want": list(range(hi - lo))}], "end": [rid] if hi == 150 else []})
+  runner = runner_for(d, dtype, 384, 64)
+  got = rc.run_in_process(runner, trace)
+  compare(got, ref, dtype, f"korurax replayed {tag}/{dtype}")
+  assert DEV == "cpu" or runner.runner.num_graphs() >= 2
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_a_request_left_out_for_many_steps_goes_on_where_it_was(korurax_dirs, dtype):
   """One request pauses in the middle of a chunk, off a page's edge, while others come, end and leave their pages; then it
   goes on with a portion of two tokens, and token by token over the chunk's end."""
