@@ -411,10 +411,10 @@ def kernel_case(name: str, reps: int = 3) -> str:
   rnd = lambda *shape, dtype=torch.bfloat16, scale=1.0: (torch.randn(*shape, generator=g, device=dev) * scale).to(dtype)
   ws = Workspace(dev)
 
-  def attention_case(dtype, page, items, **shaped):
+  def attention_case(dtype, page, items, heads=(16, 8, 128), **shaped):
     """items: (context length, new tokens) per request; the cache holds random keys and values.  ``shaped``: a cap on the
-    scores, sigmoid weights."""
-    nh, nkv, hd = 16, 8, 128
+    scores, sigmoid weights, a distance bias."""
+    nh, nkv, hd = heads
     pages_per = [-(-c // page) for c, _ in items]
     kv = rnd(sum(pages_per) + 1, 2, nkv, page, hd, dtype=dtype)
     bt = torch.zeros(len(items) + 1, max(pages_per) + 1, dtype=torch.int32)
@@ -443,8 +443,10 @@ def kernel_case(name: str, reps: int = 3) -> str:
     out = torch.empty(T, nh * hd, dtype=dtype, device=dev)
     if shaped.get("sigmoid"):
       shaped = {"softcap": shaped.get("softcap", 0.0), "score_bias": torch.full((nh,), -2.0, device=dev)}
+    elif shaped.get("distance"):
+      shaped = {"distance": torch.full((2 * nh,), 0.5, device=dev), "chunk": shaped.get("chunk")}
     return (lambda: ops.attention(out, qkv, kv, bt.to(dev), batch, nh, nkv, hd, hd ** -0.5, None, **shaped),
-            f"{len(items)} requests {items[:2]}.., page {page}, {dtype}" + (", capped scores, sigmoid weights" if shaped else ""))
+            f"{len(items)} requests {items[:2]}.., page {page}, {dtype}" + (f", scores shaped by {sorted(k for k, v in shaped.items() if v is not None)}" if shaped else ""))
 
   if name == "sample":
     R, V = 256, 151936
@@ -479,6 +481,18 @@ def kernel_case(name: str, reps: int = 3) -> str:
     fn, what = attention_case(torch.bfloat16, 64, [(2048, 2048)], softcap=50.0, sigmoid=True)       # the tcgen05 kernel on shaped scores
   elif name == "attention_decode_tma_sigmoid":
     fn, what = attention_case(torch.bfloat16, 64, [(2048 + 8 * i, 1) for i in range(64)], softcap=50.0, sigmoid=True)
+  elif name == "attention_prefill_tc_distance":
+    fn, what = attention_case(torch.bfloat16, 64, [(2048, 2048)], distance=True)
+  elif name == "attention_prefill_latent":
+    fn, what = attention_case(torch.bfloat16, 64, [(2048, 2048)], heads=(16, 1, 256))      # the mma.sync kernel, two heads a block
+  elif name == "residual_step":
+    # the end of the eighth of nine layers: 16384 rows of 2048 values - the stream, the embedding's rows and seven earlier results in
+    # float32 (1.2 GB), a bfloat16 sublayer output; the result, the averaged stream and its bfloat16 norm out
+    T, W, n = 16384, 2048, 7
+    x, first, later = (rnd(*s, dtype=torch.float32) for s in ((T, W), (T, W), (n + 1, T, W)))
+    y, res, norm_w, dw = rnd(T, W), torch.empty(T, W, dtype=torch.bfloat16, device=dev), 1 + 0.1 * rnd(W, dtype=torch.float32), rnd(n + 2, dtype=torch.float32)
+    fn = lambda: ops.residual_step(res, x, y, 0.7, x, ("layer", norm_w, None, 1e-6), None, weights=dw, first=first, later=later, n_later=n, keep=later[n])
+    what = f"{T} rows of {W}, {n} earlier layers ({T * W * ((n + 2 + 2) * 4 + 4) / 1e6:.0f} MB in and out)"
   elif name == "attention_prefill_mma":
     fn, what = attention_case(torch.bfloat16, 16, [(2048, 2048)])           # pages of 16 tokens: not the tcgen05 kernel's
   elif name == "attention_decode_cpasync":
@@ -581,7 +595,7 @@ def kernel_case(name: str, reps: int = 3) -> str:
 KERNEL_CASES = ("sample", "silu_mul", "gemm_f32", "gemm_tc_plain", "gemm_stream", "attention_generic", "attention_prefill_tc",
                 "attention_prefill_tc_pairs", "attention_prefill_mma", "attention_decode_cpasync", "experts_many_rows", "experts_few_rows",
                 "selective_scan", "delta_rule", "linear_attention", "hyper_connection", "attention_prefill_tc_sigmoid", "attention_decode_tma_sigmoid",
-                "rglru_recurrence", "mingru_recurrence")
+                "rglru_recurrence", "mingru_recurrence", "attention_prefill_tc_distance", "attention_prefill_latent", "residual_step")
 
 
 def mixed_workload(model_dir: str, requests: int = 64, outputs: int = 256) -> dict:
