@@ -49,6 +49,8 @@ constexpr int LDS = HD + 8;        // shared-memory row stride in elements (odd 
 constexpr int CHUNKS = HD / 8;     // 16-byte chunks of a row
 constexpr int KSTEPS = HD / 16;
 constexpr int NT_O = HD / 8;
+constexpr size_t SMEM_BYTES = (size_t)(16 + STAGES * 2 * BK) * LDS * sizeof(__nv_bfloat16);
+constexpr int BLOCKS_PER_SM = SMEM_BYTES <= 74 * 1024 ? 3 : (SMEM_BYTES <= 112 * 1024 ? 2 : 1);     // what shared memory leaves room for
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void cp_async16(void* dst, const void* src, bool valid) {
@@ -130,7 +132,9 @@ __device__ __forceinline__ void load_block(__nv_bfloat16* ks, __nv_bfloat16* vs,
   }
 }
 
-__global__ void __launch_bounds__(WARPS * 32, 3)
+// DISTANCE: the form for a distance bias, compiled apart so that the others carry none of it.
+template <bool DISTANCE>
+__global__ void __launch_bounds__(WARPS * 32, BLOCKS_PER_SM)
 decode_split_kernel(DecodeArgs a) {
   mi::grid_dependency_sync();
   extern __shared__ __align__(128) unsigned char smem_raw[];
@@ -185,7 +189,7 @@ decode_split_kernel(DecodeArgs a) {
     const bool shaped = a.softcap > 0.f || a.score_bias != nullptr, sigmoid = a.score_bias != nullptr;
     const float row_bias[2] = {sigmoid && g < heads ? a.score_bias[kvh * G + g0 + g] : 0.f,
                                sigmoid && g + 8 < heads ? a.score_bias[kvh * G + g0 + g + 8] : 0.f};
-    const bool distance = a.distance != nullptr;
+    constexpr bool distance = DISTANCE;
     float row_r1[2] = {0.f, 0.f}, row_r2[2] = {0.f, 0.f};
     if (distance) {
 #pragma unroll
@@ -420,7 +424,6 @@ decode_merge_kernel(DecodeArgs a) {
   }
 }
 
-constexpr size_t SMEM_BYTES = (size_t)(16 + STAGES * 2 * BK) * LDS * sizeof(__nv_bfloat16);
 static_assert((size_t)WARPS * 16 * HD * 4 + WARPS * 16 * 2 * 4 <= (size_t)STAGES * 2 * BK * LDS * 2,
               "the warps' results must fit into the stages");
 
@@ -470,13 +473,14 @@ MI_API int mi_attention_decode_bf16(void* out, const void* q_base, int q_stride,
   a.softcap = softcap; a.score_bias = score_bias; a.gate_per_head = gate_per_head; a.distance = distance;
   static bool configured = false;
   if (!configured) {
-    cudaError_t err = cudaFuncSetAttribute(decode_split_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);
+    cudaError_t err = cudaFuncSetAttribute(decode_split_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);
+    if (err == cudaSuccess) err = cudaFuncSetAttribute(decode_split_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);
     if (err != cudaSuccess) return mi_fail("attention_decode: cannot get %zu bytes of shared memory: %s", SMEM_BYTES, cudaGetErrorString(err));
     configured = true;
   }
   // more than eight query heads on a kv head: the merge as a kernel of its own, a block per (request, head)
   a.merge_apart = nh / nkv > 8 ? 1 : 0;
-  mi::launch(decode_split_kernel, dim3(dim3(nkv, max_splits, n_dec)), dim3(WARPS * 32), SMEM_BYTES, stream, a);
+  mi::launch(distance ? decode_split_kernel<true> : decode_split_kernel<false>, dim3(dim3(nkv, max_splits, n_dec)), dim3(WARPS * 32), SMEM_BYTES, stream, a);
   if (a.merge_apart) mi::launch(decode_merge_kernel, dim3(nh, n_dec), dim3(128), 0, stream, a);
   MI_LAUNCH_OK("attention_decode");
   return 0;

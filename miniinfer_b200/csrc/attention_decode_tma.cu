@@ -115,6 +115,8 @@ __device__ __forceinline__ bool consumer_any(bool flag) {
       : "=r"(out) : "r"((uint32_t)flag), "n"(CONSUMERS * 32) : "memory");
   return out != 0;
 }
+// DISTANCE: the form for a distance bias, compiled apart so that the others carry none of it.
+template <bool DISTANCE>
 __global__ void __launch_bounds__(THREADS, 1)
 decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map, Args a) {
   extern __shared__ __align__(1024) unsigned char smem_raw[];
@@ -419,7 +421,7 @@ decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map, Args a) {
 #pragma unroll
         for (int c = 0; c < 4; ++c) o[i][c] = 0.f;
       float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};   // heads 2t and 2t + 1
-      const TileScores shape = tile_scores(a.scale, a.softcap, a.score_bias, a.distance, a.nh, d.kvh * G + g0 + 2 * t4, heads - 2 * t4, d.pos);
+      const TileScores shape = tile_scores(a.scale, a.softcap, a.score_bias, DISTANCE ? a.distance : nullptr, a.nh, d.kvh * G + g0 + 2 * t4, heads - 2 * t4, d.pos);
 
       // tile gb of this block's stream goes to warp gb mod 3 (it owns the stages gb mod `stages` can be);
       // `rank` is the warp's place among the item's tiles, which fixes the order of the merge
@@ -590,7 +592,8 @@ MI_API int mi_attention_decode_tma(void* out, const void* q_base, int q_stride, 
   const size_t smem = smem_bytes(stages, a.gp, max_splits, n_dec);
   static size_t configured = 0;
   if (smem > configured) {
-    cudaError_t err = cudaFuncSetAttribute(decode_tma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    cudaError_t err = cudaFuncSetAttribute(decode_tma_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    if (err == cudaSuccess) err = cudaFuncSetAttribute(decode_tma_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
     if (err != cudaSuccess) return mi_fail("attention_decode_tma: cannot get shared memory: %s", cudaGetErrorString(err));
     configured = 227 * 1024;
   }
@@ -598,7 +601,7 @@ MI_API int mi_attention_decode_tma(void* out, const void* q_base, int q_stride, 
   memcpy(&map, kv_map, sizeof(map));
   MI_REQUIRE(n_dec <= 4096, "attention_decode_tma: at most 4096 decode entries per launch (got %d)", n_dec);
   const int grid = num_sms;
-  mi::launch(decode_tma_kernel, dim3(grid), dim3(THREADS), smem, stream, map, a);
+  mi::launch(distance ? decode_tma_kernel<true> : decode_tma_kernel<false>, dim3(grid), dim3(THREADS), smem, stream, map, a);
   MI_LAUNCH_OK("attention_decode_tma");
   return 0;
 }
