@@ -72,6 +72,20 @@ class CompositeSpec:
 CacheSpec = Union[PagedKVSpec, FixedStateSpec, CompositeSpec]
 
 
+def shared_need(specs) -> CacheSpec:
+  """The need of one cache that several layers read: keys and values of one shape for as long as any of them can see them -
+  the widest window, or everything once a reader sees every earlier key or the readers mix windows and chunks.
+  ``ValueError`` if the layers differ in what a row holds."""
+  first = specs[0]
+  if all(s == first for s in specs):
+    return first
+  if not all(isinstance(s, PagedKVSpec) and (s.num_kv_heads, s.head_dim) == (first.num_kv_heads, first.head_dim) for s in specs):
+    raise ValueError("layers that share a cache differ in what they keep in it")
+  windows = [s.window for s in specs]
+  if all(w is not None for w in windows):
+    return PagedKVSpec(first.num_kv_heads, first.head_dim, max(windows), max(s.keep_first for s in specs))
+  return PagedKVSpec(first.num_kv_heads, first.head_dim)
+
 
 def flatten_specs(layer_specs):
   """The needs of all layers, the members of composite ones one by one, without the layers that keep nothing."""

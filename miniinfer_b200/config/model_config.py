@@ -957,3 +957,131 @@ class KoruraxConfig(ModelConfig):
          "residual_mult": self.residual_mult, "logit_softcap": self.logit_softcap, "layers": [dict(x) for x in self.layers]}
     d.update(self.extra)
     return d
+
+
+@dataclass
+class WindowedLatentConfig(LatentAttentionConfig):
+  """``layers[i].mixer`` of a Besolix ``latent_attention`` layer.  ``window``: ``mask.size``; ``kv_from``: the earlier layer whose
+  latents and rotated key parts this layer reads instead of keeping its own."""
+
+  window: Optional[int] = None
+  kv_from: Optional[int] = None
+
+
+@dataclass
+class RotatedWindowAttentionConfig:
+  """``layers[i].mixer`` of a Besolix ``attention`` layer: grouped-query attention with normed, rotated heads over the last
+  ``window`` positions (``mask.size``; None: every earlier one)."""
+
+  heads: int
+  kv_heads: int
+  dim: int
+  vdim: int
+  scale: float
+  window: Optional[int]
+  rot: RotationConfig
+
+
+@dataclass
+class BesolixConfig(ModelConfig):
+  """Besolix: a decoder whose layers are listed one by one (``layers[i].{type, mixer, mlp}``), each a pre-norm layer (RMS norms
+  stored around zero) of a mixer and a dense feed-forward gated by a tanh GELU (or none); mixers of three types -
+  ``latent_attention`` (windowed, with a gate a value; a layer with ``mixer.kv_from: j`` reads layer ``j``'s latents),
+  ``attention`` (windowed grouped-query attention, frequencies divided by ``rot.scaling.factor``) and ``delta`` (a gated delta
+  rule with one decay a head).  The head is a matrix of its own.  Other keys: ``architecture``, ``vocab``, ``width``,
+  ``norm.eps``.  The design has no position limit of its own; ``max_position_embeddings`` is only the engine's bound."""
+
+  architecture: str = "Besolix"
+  vocab: int = 0
+  width: int = 0
+  norm: Dict[str, Any] = field(default_factory=dict)
+  layers: List[Dict[str, Any]] = field(default_factory=list)
+  max_position_embeddings: int = 1 << 30
+  initializer_range: float = 0.02
+
+  TYPES = ("latent_attention", "attention", "delta")
+
+  def validate(self) -> None:
+    if not self.architectures:
+      self.architectures = [self.architecture]
+    self.vocab_size = self.vocab
+    for key in ("vocab", "width"):
+      v = getattr(self, key)
+      if not isinstance(v, int) or isinstance(v, bool) or v <= 0:
+        raise ConfigError(f"{key} must be a positive integer, got {v!r}")
+    eps = self.norm.get("eps") if isinstance(self.norm, dict) else None
+    if not isinstance(eps, (int, float)) or isinstance(eps, bool) or not eps > 0:
+      raise ConfigError(f"norm.eps must be a positive number, got {eps!r}")
+    if not self.layers:
+      raise ConfigError("layers must list at least one layer")
+    for i in range(len(self.layers)):
+      self.mixer_of(i)
+      self.ff_of(i)
+
+  @property
+  def norm_eps(self) -> float:
+    return float(self.norm["eps"])
+
+  def type_of(self, i: int) -> str:
+    kind = self.layers[i].get("type")
+    if kind not in self.TYPES:
+      raise ConfigError(f"layers[{i}].type={kind!r} is not a mixer of this design (known: {', '.join(self.TYPES)})")
+    return kind
+
+  def mixer_of(self, i: int):
+    """The typed mixer configuration of layer ``i``: a ``WindowedLatentConfig``, a ``RotatedWindowAttentionConfig`` or a
+    ``GatedDeltaConfig``."""
+    kind = self.type_of(i)
+    m = self.layers[i].get("mixer")
+    where = f"layers[{i}].mixer"
+    if not isinstance(m, dict):
+      raise ConfigError(f"{where} is missing")
+    if kind == "delta":
+      d = GatedDeltaConfig(*(_positive_int(m, k, where) for k in ("heads", "kv_heads", "dim", "vdim", "conv")))
+      if d.heads % d.kv_heads:
+        raise ConfigError(f"{where}.heads={d.heads} must be a multiple of kv_heads={d.kv_heads}")
+      return d
+    mask = m.get("mask")
+    window = None
+    if mask is not None:
+      if not isinstance(mask, dict):
+        raise ConfigError(f"{where}.mask must be an object")
+      window = _positive_int(mask, "size", where + ".mask")
+    rot = RotationConfig.read(m, where, ("factor",))
+    if kind == "attention":
+      a = RotatedWindowAttentionConfig(*(_positive_int(m, k, where) for k in ("heads", "kv_heads", "dim", "vdim")),
+                                       _number(m, "scale", where), window, rot)
+      if a.heads % a.kv_heads:
+        raise ConfigError(f"{where}.heads={a.heads} must be a multiple of kv_heads={a.kv_heads}")
+      if rot.dims > a.dim:
+        raise ConfigError(f"{where}.rot.dims={rot.dims} is more than dim={a.dim}")
+      return a
+    c = WindowedLatentConfig(*(_positive_int(m, k, where) for k in ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank")),
+                             _number(m, "scale", where), rot, window, m.get("kv_from"))
+    if rot.dims != c.rot_dim:
+      raise ConfigError(f"{where}.rot.dims={rot.dims} must equal rot_dim={c.rot_dim}: the rotated part is rotated whole")
+    if c.kv_from is not None:
+      j = c.kv_from
+      if not isinstance(j, int) or isinstance(j, bool) or not (0 <= j < i) or self.layers[j].get("type") != "latent_attention":
+        raise ConfigError(f"{where}.kv_from={j!r} must name an earlier latent_attention layer")
+      src = self.mixer_of(j)
+      if src.kv_from is not None:
+        raise ConfigError(f"{where}.kv_from={j} names a layer that keeps no latents of its own")
+      if (src.kv_rank, src.rot_dim, src.rot) != (c.kv_rank, c.rot_dim, c.rot):
+        raise ConfigError(f"{where}.kv_from={j}: kv_rank, rot_dim and rot must equal those of layers[{j}]")
+    return c
+
+  def ff_of(self, i: int) -> Optional[int]:
+    """The width of layer ``i``'s dense feed-forward, or None for a layer without one."""
+    mlp = self.layers[i].get("mlp")
+    if mlp is None:
+      return None
+    if not isinstance(mlp, dict) or mlp.get("kind") != "dense":
+      raise ConfigError(f"layers[{i}].mlp.kind={mlp.get('kind') if isinstance(mlp, dict) else mlp!r} is not known (dense)")
+    return _positive_int(mlp, "ff", f"layers[{i}].mlp")
+
+  def to_dict(self) -> Dict[str, Any]:
+    d = {"architecture": self.architecture, "vocab": self.vocab, "width": self.width, "norm": dict(self.norm),
+         "layers": [dict(x) for x in self.layers]}
+    d.update(self.extra)
+    return d

@@ -120,7 +120,7 @@ MI_API int mi_softcap(float* x, long long n, float cap, cudaStream_t stream) {
 // kind: a MiGlu; limit: the clamp of MI_GLU_CLAMPED.
 MI_API int mi_glu_mul(void* out, const void* gu, int dtype, int T, int I, int kind, float limit, cudaStream_t stream) {
   MI_REQUIRE(T >= 0 && I > 0, "glu_mul: bad sizes T=%d I=%d", T, I);
-  MI_REQUIRE(kind == MI_GLU_SILU || (kind == MI_GLU_CLAMPED && limit > 0.f), "glu_mul: unknown kind %d or a limit that is not positive", kind);
+  MI_REQUIRE(mi_glu_known(kind, limit), "glu_mul: unknown kind %d or a limit that is not positive", kind);
   if (T == 0) return 0;
   const size_t total = (size_t)T * I;
   const int threads = 256;

@@ -18,7 +18,10 @@
 #define MI_API extern "C" __attribute__((visibility("default")))
 
 enum MiDtype { MI_F32 = 0, MI_BF16 = 1 };
-enum MiGlu { MI_GLU_SILU = 0, MI_GLU_CLAMPED = 1 };   // gated activations: see mi::glu_fast
+enum MiGlu { MI_GLU_SILU = 0, MI_GLU_CLAMPED = 1, MI_GLU_GELU_TANH = 2 };   // gated activations: see mi::glu_fast
+inline bool mi_glu_known(int glu, float limit) {
+  return glu == MI_GLU_SILU || glu == MI_GLU_GELU_TANH || (glu == MI_GLU_CLAMPED && limit > 0.f);
+}
 
 inline thread_local char mi_error_text[1024] = "";
 
@@ -107,12 +110,18 @@ __device__ __forceinline__ float silu_mul_exact(float g, float u) { return g / (
 // The gated activations of the feed-forwards, act(g) * u from a gate value g and an up value u (MiGlu):
 //   MI_GLU_SILU     silu(g) * u
 //   MI_GLU_CLAMPED  with a limit L: g' = min(g, L), u' = clamp(u, -L, L); g' * sigmoid(1.702 g') * (u' + 1)
+//   MI_GLU_GELU_TANH  g / 2 * (1 + tanh(y)) * u with y = sqrt(2 / pi) (g + 0.044715 g^3)
+// (the fast form of the last as g * sigmoid(2 y), which it equals; the exponent stays where the exponential is finite).
 // `fast` forms for the bfloat16 paths (hardware exponential and reciprocal), `exact` ones for float32.
 __device__ __forceinline__ float glu_fast(float g, float u, int kind, float limit) {
   if (kind == MI_GLU_CLAMPED) {
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
     return __fdividef(g, 1.f + __expf(-1.702f * g)) * (u + 1.f);
+  }
+  if (kind == MI_GLU_GELU_TANH) {
+    const float y = 0.7978845608028654f * fmaf(0.044715f * g * g, g, g);
+    return __fdividef(g, 1.f + __expf(fminf(-2.f * y, 80.f))) * u;
   }
   return silu_mul_fast(g, u);
 }
@@ -122,6 +131,7 @@ __device__ __forceinline__ float glu_exact(float g, float u, int kind, float lim
     u = fminf(fmaxf(u, -limit), limit);
     return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
   }
+  if (kind == MI_GLU_GELU_TANH) return 0.5f * g * (1.f + tanhf(0.7978845608028654f * fmaf(0.044715f * g * g, g, g))) * u;
   return silu_mul_exact(g, u);
 }
 

@@ -1,13 +1,14 @@
 // A batch of small matrix products over strided operands, for any sizes and alignments:
 //
-//   out[b][m, n] = act( sum_k x[b][m, k] * w[b][n, k]  (+ bias[n]) )  (* sigmoid(row_gate[m, b]))
+//   out[b][m, n] = act( sum_k x[b][m, k] * w[b][n, k]  (+ bias[n]) )  (* sigmoid(row_gate[m, b]) or * sigmoid(value_gate[m, b N + n]))
 //
 // x[b] starts at x + b * x_batch with rows lda apart, w[b] at w + b * w_batch with rows ldw apart, out[b] at
 // out + b * o_batch with rows ldo apart - so the heads of a token's row (a batch stride of one head, a row stride of
 // the whole row) are multiplied with a matrix per head without being repacked, and a column range of a row can be
 // an operand.  Products and sums in float32, k ascending, whatever the storage type: a row's result does not depend
 // on the other rows.  act: 0 none, 1 softplus (log(1 + exp(z)), z itself above 20).  row_gate: one logit per
-// (row, batch) at row_gate[m * gate_stride + b]; the output rows of batch b are multiplied with its sigmoid.
+// (row, batch) at row_gate[m * gate_stride + b]; the output rows of batch b are multiplied with its sigmoid.  value_gate: one
+// logit per output value instead, at value_gate[m * gate_stride + b * N + n].
 //
 // This is the product of the 32-bit path for strided operands, of per-head up- and down-projections of a latent
 // attention, and the fallback of the bfloat16 path for inner sizes that are no multiple of 8.  Tiles of 64 x 64
@@ -27,6 +28,7 @@ struct BatchedArgs {
   int act;
   const void* row_gate;
   int gate_stride;
+  const void* value_gate;      // one logit per output value: row m at m * gate_stride, batch b's N values from column b * N on
 };
 
 template <typename T, typename TO>
@@ -82,6 +84,7 @@ gemm_batched_kernel(BatchedArgs a) {
       float y = acc[i][j];
       if (a.bias) y += a.bias[n];
       if (a.act == 1) y = y > 20.f ? y : log1pf(expf(y));
+      if (a.value_gate) y *= 1.f / (1.f + expf(-mi::to_float(((const T*)a.value_gate)[(size_t)m * a.gate_stride + (size_t)b * a.N + n])));
       out[(size_t)m * a.ldo + n] = mi::from_float<TO>(y * gate);
     }
   }
@@ -121,6 +124,7 @@ gemm_batched_few_rows_kernel(BatchedArgs a) {
       if (a.bias) y += a.bias[n];
       if (a.act == 1) y = y > 20.f ? y : log1pf(expf(y));
       if (a.row_gate) y *= 1.f / (1.f + expf(-__bfloat162float(((const __nv_bfloat16*)a.row_gate)[(size_t)m * a.gate_stride + b])));
+      if (a.value_gate) y *= 1.f / (1.f + expf(-__bfloat162float(((const __nv_bfloat16*)a.value_gate)[(size_t)m * a.gate_stride + (size_t)b * a.N + n])));
       out[(size_t)m * a.ldo + n] = mi::from_float<TO>(y);
     }
   }
@@ -130,14 +134,14 @@ gemm_batched_few_rows_kernel(BatchedArgs a) {
 
 MI_API int mi_gemm_batched_few_rows(void* out, int out_dtype, const void* x, const void* w, int dtype, int batch, int M, int N, int K,
                                     int lda, long long x_batch, int ldw, long long w_batch, int ldo, long long o_batch,
-                                    const float* bias, int act, const void* row_gate, int gate_stride, cudaStream_t stream) {
+                                    const float* bias, int act, const void* row_gate, int gate_stride, const void* value_gate, cudaStream_t stream) {
   MI_REQUIRE(batch > 0 && batch <= 65535 && M >= 0 && M <= FEW_ROWS && N > 0 && K > 0, "gemm_batched_few_rows: bad sizes batch=%d M=%d N=%d K=%d", batch, M, N, K);
   MI_REQUIRE(dtype == MI_BF16 && lda >= K && ldw >= K && ldo >= N && (act == 0 || act == 1), "gemm_batched_few_rows: bfloat16 operands, rows that do not overlap");
   if (M == 0) return 0;
   BatchedArgs a;
   a.x = x; a.w = w; a.out = out; a.x_batch = x_batch; a.w_batch = w_batch; a.o_batch = o_batch;
   a.lda = lda; a.ldw = ldw; a.ldo = ldo; a.M = M; a.N = N; a.K = K; a.bias = bias; a.act = act;
-  a.row_gate = row_gate; a.gate_stride = gate_stride;
+  a.row_gate = row_gate; a.gate_stride = gate_stride; a.value_gate = value_gate;
   dim3 grid((N + 3) / 4, batch);
   if (out_dtype == MI_BF16) mi::launch(gemm_batched_few_rows_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, a);
   else if (out_dtype == MI_F32) mi::launch(gemm_batched_few_rows_kernel<float>, grid, dim3(128), 0, stream, a);
@@ -148,15 +152,16 @@ MI_API int mi_gemm_batched_few_rows(void* out, int out_dtype, const void* x, con
 
 MI_API int mi_gemm_batched(void* out, int out_dtype, const void* x, const void* w, int dtype, int batch, int M, int N, int K,
                            int lda, long long x_batch, int ldw, long long w_batch, int ldo, long long o_batch,
-                           const float* bias, int act, const void* row_gate, int gate_stride, cudaStream_t stream) {
+                           const float* bias, int act, const void* row_gate, int gate_stride, const void* value_gate, cudaStream_t stream) {
   MI_REQUIRE(batch > 0 && batch <= 65535 && M >= 0 && N > 0 && K > 0, "gemm_batched: bad sizes batch=%d M=%d N=%d K=%d", batch, M, N, K);
   MI_REQUIRE(lda >= K && ldw >= K && ldo >= N, "gemm_batched: rows overlap (lda=%d ldw=%d ldo=%d)", lda, ldw, ldo);
   MI_REQUIRE(act == 0 || act == 1, "gemm_batched: unknown activation %d", act);
+  MI_REQUIRE(row_gate == nullptr || value_gate == nullptr, "gemm_batched: a gate a row or a gate a value, not both");
   if (M == 0) return 0;
   BatchedArgs a;
   a.x = x; a.w = w; a.out = out; a.x_batch = x_batch; a.w_batch = w_batch; a.o_batch = o_batch;
   a.lda = lda; a.ldw = ldw; a.ldo = ldo; a.M = M; a.N = N; a.K = K; a.bias = bias; a.act = act;
-  a.row_gate = row_gate; a.gate_stride = gate_stride;
+  a.row_gate = row_gate; a.gate_stride = gate_stride; a.value_gate = value_gate;
   dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM, batch);
   MI_REQUIRE(grid.y <= 65535, "gemm_batched: M=%d is too large for one launch", M);
   if (dtype == MI_F32 && out_dtype == MI_F32) mi::launch(gemm_batched_kernel<float, float>, grid, dim3(256), 0, stream, a);
@@ -164,5 +169,48 @@ MI_API int mi_gemm_batched(void* out, int out_dtype, const void* x, const void* 
   else if (dtype == MI_BF16 && out_dtype == MI_F32) mi::launch(gemm_batched_kernel<__nv_bfloat16, float>, grid, dim3(256), 0, stream, a);
   else return mi_fail("gemm_batched: unsupported dtypes operands=%d out=%d", dtype, out_dtype);
   MI_LAUNCH_OK("gemm_batched");
+  return 0;
+}
+
+namespace {
+// x[m, i] *= sigmoid(gate[m, i]) over bfloat16 rows, 8 values a thread where the rows are 16-byte aligned.
+template <int V>
+__global__ void __launch_bounds__(256)
+sigmoid_gate_kernel(__nv_bfloat16* __restrict__ x, long long ldx, const __nv_bfloat16* __restrict__ gate, long long ldg, int N, size_t total) {
+  mi::grid_dependency_sync();
+  const int per_row = N / V;
+  for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
+    const size_t m = idx / per_row;
+    const int i = (int)(idx - m * per_row) * V;
+    __nv_bfloat16* xp = x + m * ldx + i;
+    const __nv_bfloat16* gp = gate + m * ldg + i;
+    if (V == 8) {
+      uint4 xv = *reinterpret_cast<const uint4*>(xp);
+      const uint4 gv = *reinterpret_cast<const uint4*>(gp);
+      __nv_bfloat162* xs = reinterpret_cast<__nv_bfloat162*>(&xv);
+      const __nv_bfloat162* gs = reinterpret_cast<const __nv_bfloat162*>(&gv);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float2 a = __bfloat1622float2(xs[k]), g = __bfloat1622float2(gs[k]);
+        xs[k] = __floats2bfloat162_rn(__fdividef(a.x, 1.f + __expf(-g.x)), __fdividef(a.y, 1.f + __expf(-g.y)));
+      }
+      *reinterpret_cast<uint4*>(xp) = xv;
+    } else {
+      *xp = __float2bfloat16_rn(__fdividef(__bfloat162float(*xp), 1.f + __expf(-__bfloat162float(*gp))));
+    }
+  }
+}
+}  // namespace
+
+// x [M, N] *= sigmoid(gate [M, N]), bfloat16, in place; rows ldx and ldg values apart.
+MI_API int mi_sigmoid_gate_bf16(void* x, long long ldx, const void* gate, long long ldg, int M, int N, cudaStream_t stream) {
+  MI_REQUIRE(M >= 0 && N > 0 && ldx >= N && ldg >= N, "sigmoid_gate: bad sizes M=%d N=%d", M, N);
+  if (M == 0) return 0;
+  const bool vec = N % 8 == 0 && ldx % 8 == 0 && ldg % 8 == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)gate % 16) == 0;
+  const size_t total = (size_t)M * N / (vec ? 8 : 1), want = (total + 255) / 256, most = (size_t)mi::sm_count() * 16;
+  const dim3 grid((unsigned)(want < most ? want : most));
+  if (vec) mi::launch(sigmoid_gate_kernel<8>, grid, dim3(256), 0, stream, (__nv_bfloat16*)x, ldx, (const __nv_bfloat16*)gate, ldg, N, total);
+  else mi::launch(sigmoid_gate_kernel<1>, grid, dim3(256), 0, stream, (__nv_bfloat16*)x, ldx, (const __nv_bfloat16*)gate, ldg, N, total);
+  MI_LAUNCH_OK("sigmoid_gate");
   return 0;
 }

@@ -21,7 +21,7 @@ MI_API int mi_gemm_skinny_glu_bf16(void* out, const void* x, const void* w, int 
   MI_REQUIRE(I > 0 && K > 0 && ldo >= I, "gemm_skinny_glu: bad sizes I=%d K=%d ldo=%d", I, K, ldo);
   MI_REQUIRE(K % 8 == 0, "gemm_skinny_glu: K=%d must be a multiple of 8 (16-byte loads of bf16 rows)", K);
   MI_REQUIRE(((uintptr_t)x % 16) == 0 && ((uintptr_t)w % 16) == 0, "gemm_skinny_glu: operands must be 16-byte aligned");
-  MI_REQUIRE(glu == MI_GLU_SILU || (glu == MI_GLU_CLAMPED && limit > 0.f), "gemm_skinny_glu: unknown activation %d or a limit that is not positive", glu);
+  MI_REQUIRE(mi_glu_known(glu, limit), "gemm_skinny_glu: unknown activation %d or a limit that is not positive", glu);
   if (M == 0) return 0;
   FuseArgs fa{nullptr, nullptr, 0.f};
   fa.glu = glu;

@@ -214,7 +214,8 @@ struct Walk {
 // mma.sync kernel: 0.868 ms).
 __device__ __forceinline__ void dep_sync() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 
-template <bool SWIGLU, typename TOut>
+// GLU: the gated activation of the SWIGLU form (a MiGlu of common.cuh that takes no limit).
+template <bool SWIGLU, typename TOut, int GLU = MI_GLU_SILU>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_stream_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant__ CUtensorMap w_map, Args a) {
   // The stages are read in the 128-byte swizzle, whose pattern repeats every 1024 bytes of address: the kernel has no
@@ -402,7 +403,7 @@ gemm_stream_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_co
             if (n < a.N && ok) {
 #pragma unroll
               for (int m = 0; m < NB; ++m)
-                if (m < a.M) store_out<TOut>(out + (size_t)m * a.ldo + n, mi::silu_mul_fast(round_bf16(v[m]), round_bf16(up_s[r * NB + m])));
+                if (m < a.M) store_out<TOut>(out + (size_t)m * a.ldo + n, mi::glu_fast(round_bf16(v[m]), round_bf16(up_s[r * NB + m]), GLU, 0.f));
             }
           }
           asm volatile("bar.sync 1, %0;" ::"n"(EPILOGUE_WARPS * 32) : "memory");   // up_s may be written again
@@ -453,7 +454,7 @@ int encode_map(CUtensorMap* map, const void* base, long long rows, long long col
   return 0;
 }
 
-template <bool SWIGLU, typename TOut>
+template <bool SWIGLU, typename TOut, int GLU = MI_GLU_SILU>
 int run(void* out, const void* x, const void* w, int M, int N, int K, int ldo, float* parts, int* counters, int counters_len,
         int parts_blocks, int* status, cudaStream_t stream) {
   MI_REQUIRE(M > 0 && M <= NB && N > 0 && K >= BK && K % 8 == 0 && ldo >= N,
@@ -477,7 +478,7 @@ int run(void* out, const void* x, const void* w, int M, int N, int K, int ldo, f
   CUtensorMap xm, wm;
   if (int e = encode_map(&xm, x, M, K, NB)) return e;
   if (int e = encode_map(&wm, w, SWIGLU ? 2LL * N : (long long)N, K, HALF_ROWS)) return e;
-  auto kernel = gemm_stream_tc_kernel<SWIGLU, TOut>;
+  auto kernel = gemm_stream_tc_kernel<SWIGLU, TOut, GLU>;
   static bool configured = false;
   if (!configured) {
     cudaError_t err = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);
@@ -512,4 +513,10 @@ MI_API int mi_gemm_stream_tc_bf16(void* out, int out_dtype, const void* x, const
 MI_API int mi_gemm_stream_tc_swiglu_bf16(void* out, const void* x, const void* w, int M, int I, int K, int ldo,
                                          float* parts, int* counters, int counters_len, int parts_blocks, int* status, cudaStream_t stream) {
   return run<true, __nv_bfloat16>(out, x, w, M, I, K, ldo, parts, counters, counters_len, parts_blocks, status, stream);
+}
+
+// out[M, I] = gelu_tanh(x w[0:I]^T) * (x w[I:2I]^T), all bf16.
+MI_API int mi_gemm_stream_tc_geglu_bf16(void* out, const void* x, const void* w, int M, int I, int K, int ldo,
+                                        float* parts, int* counters, int counters_len, int parts_blocks, int* status, cudaStream_t stream) {
+  return run<true, __nv_bfloat16, MI_GLU_GELU_TANH>(out, x, w, M, I, K, ldo, parts, counters, counters_len, parts_blocks, status, stream);
 }

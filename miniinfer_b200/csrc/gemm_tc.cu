@@ -548,8 +548,9 @@ MI_API int mi_gemm_tc_swiglu_bf16(void* out, const void* x, const void* w, int M
 // The same with another gated activation (a MiGlu of common.cuh) in the epilogue.
 MI_API int mi_gemm_tc_glu_bf16(void* out, const void* x, const void* w, int M, int I, int K, int ldo, int* status,
                                int pairs, int glu, float limit, cudaStream_t stream) {
-  MI_REQUIRE(glu == MI_GLU_SILU || (glu == MI_GLU_CLAMPED && limit > 0.f), "gemm_tc_glu: unknown activation %d or a limit that is not positive", glu);
+  MI_REQUIRE(mi_glu_known(glu, limit), "gemm_tc_glu: unknown activation %d or a limit that is not positive", glu);
   if (glu == MI_GLU_CLAMPED) return run<true, false, MI_GLU_CLAMPED>(out, x, w, M, I, K, ldo, status, pairs, stream, 1, nullptr, 0, 0, glu, limit);
+  if (glu == MI_GLU_GELU_TANH) return run<true, false, MI_GLU_GELU_TANH>(out, x, w, M, I, K, ldo, status, pairs, stream, 1, nullptr, 0, 0, glu, limit);
   return run<true>(out, x, w, M, I, K, ldo, status, pairs, stream);
 }
 
@@ -560,11 +561,13 @@ MI_API int mi_gemm_tc_glu_bf16(void* out, const void* x, const void* w, int M, i
 // written instead of the product.
 MI_API int mi_gemm_tc_grouped_bf16(void* out, const void* x, const void* w, int M, int N, int K, int ldo, int experts, int swiglu,
                                    const int* tile_expert, int tile_rows, int* status, int pairs, int glu, float limit, int relu2, cudaStream_t stream) {
-  MI_REQUIRE(glu == MI_GLU_SILU || (glu == MI_GLU_CLAMPED && limit > 0.f), "gemm_tc_grouped: unknown activation %d or a limit that is not positive", glu);
+  MI_REQUIRE(mi_glu_known(glu, limit), "gemm_tc_grouped: unknown activation %d or a limit that is not positive", glu);
   MI_REQUIRE(experts > 0 && tile_expert != nullptr && tile_rows > 0 && tile_rows % 256 == 0 && M % tile_rows == 0,
              "gemm_tc_grouped: rows=%d must come in stretches of tile_rows=%d, a multiple of 256", M, tile_rows);
   if (swiglu && glu == MI_GLU_CLAMPED)
     return run<true, true, MI_GLU_CLAMPED>(out, x, w, M, N, K, ldo, status, pairs, stream, experts, tile_expert, tile_rows, 0, glu, limit);
+  if (swiglu && glu == MI_GLU_GELU_TANH)
+    return run<true, true, MI_GLU_GELU_TANH>(out, x, w, M, N, K, ldo, status, pairs, stream, experts, tile_expert, tile_rows, 0, glu, limit);
   return swiglu ? run<true, true>(out, x, w, M, N, K, ldo, status, pairs, stream, experts, tile_expert, tile_rows)
                 : run<false, true>(out, x, w, M, N, K, ldo, status, pairs, stream, experts, tile_expert, tile_rows, relu2 ? 1 : 0);
 }

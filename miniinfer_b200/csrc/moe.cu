@@ -552,7 +552,7 @@ MI_API int mi_moe_align(const int* topk_idx, int n_pairs, int E, int TM, int* so
 MI_API int mi_moe_gemm(const void* a_rows, int dtype, int a_stride, const void* w, void* out, const int* sorted_pair,
                        const int* tile_expert, int max_tiles, int TM, int N, int K, int top, int mode, int glu, float limit,
                        cudaStream_t stream) {
-  MI_REQUIRE(glu == MI_GLU_SILU || (glu == MI_GLU_CLAMPED && limit > 0.f), "moe_gemm: unknown activation %d or a limit that is not positive", glu);
+  MI_REQUIRE(mi_glu_known(glu, limit), "moe_gemm: unknown activation %d or a limit that is not positive", glu);
   MI_REQUIRE(mode >= PLAIN && mode <= ACTIVATED, "moe_gemm: unknown mode %d", mode);
   MI_REQUIRE(N > 0 && K > 0 && max_tiles >= 0 && max_tiles <= 65535, "moe_gemm: bad sizes N=%d K=%d tiles=%d", N, K, max_tiles);
   if (max_tiles == 0) return 0;

@@ -9,6 +9,8 @@
 // result at a position does not depend on how the request was cut into steps or on what else is in the batch.  All
 // arithmetic of the recurrences - decays, their logarithms, softplus, exponentials, step sizes, gates, unit norms,
 // the state and the sums over it - is float32; activations are read and written in the storage type.
+#include <type_traits>
+
 #include "common.cuh"
 
 namespace {
@@ -281,7 +283,11 @@ scan_carry_kernel(float* __restrict__ seg_state, const float* __restrict__ seg_d
 //   qh = q / sqrt(sum q^2 + 1e-6) * dim^-1/2,  kh = k / sqrt(sum k^2 + 1e-6)       (q, k of the head's q/k head)
 //   g[i] = exp(-exp(A_log[head]) * softplus(a[t, head, i] + dt_bias[head, i])),    beta = sigmoid(b[t, head])
 //   S[i, :] <- g[i] * S[i, :];   u = beta * (v - S^T kh);   S <- S + kh u^T;   o = S^T qh
-//   out[t, head, :] = o / sqrt(mean(o^2) + eps) * norm_w * sigmoid(gate[t, head, :])
+//   out[t, head, :] = o / sqrt(mean(o^2) + eps) * norm_w * sigmoid(gate[t, head, :])   (or silu of the gate)
+// With one decay a head (HEAD_DECAY) a[t, head] and dt_bias[head] stand for a row of them.  The decay is then a number that
+// multiplies the whole state, so kh and qh can both be read against the state as the token finds it,
+//   S^T kh before the write = g (S_old^T kh),      o = g (S_old^T qh) + (qh . kh) u,
+// and the two sums over a column run side by side instead of one behind the other.
 // Three kernels.  (1) delta_prepare, a warp per (token, head), all tokens at once: everything of a token that does not
 // depend on the state - unit q and k, decays, beta - as float32 rows.  (2) delta_recurrence, the only part that walks
 // the tokens in order: a block per (item, head, group of value columns).  Thread (j, r) keeps rows r * DK .. r * DK + DK - 1
@@ -296,7 +302,9 @@ struct DeltaPrepArgs {
   const T* b; int ldb;                   // beta logits, head h at column h
   const float* dt_bias; const float* A_log;
   float* qn; float* kn;                  // [tokens, kv_heads * dim]
-  float* g;                              // [tokens, heads * dim]
+  float* g;                              // [tokens, heads * dim], or [tokens, heads] with one decay a head
+  float* qk;                             // [tokens, kv_heads]: qh . kh (one decay a head only)
+  int head_decay;
   float* beta;                           // [tokens, heads]
   const T* v; int ldv;                   // values, head h at column h * vdim
   float* raw;                            // [tokens, heads * vdim]: receives the values as float32 (the recurrence reads a
@@ -324,14 +332,23 @@ delta_prepare_kernel(DeltaPrepArgs<T> a) {
       sq = mi::warp_sum(sq);
       sk = mi::warp_sum(sk);
       const float fq = rsqrtf((float)a.dim) / sqrtf(sq + 1e-6f), fk = 1.f / sqrtf(sk + 1e-6f);
+      float qk = 0.f;
       for (int i = lane; i < a.dim; i += 32) {
-        a.qn[((size_t)t * a.kv_heads + u) * a.dim + i] = mi::to_float(q[i]) * fq;
-        a.kn[((size_t)t * a.kv_heads + u) * a.dim + i] = mi::to_float(k[i]) * fk;
+        const float qv = mi::to_float(q[i]) * fq, kv = mi::to_float(k[i]) * fk;
+        a.qn[((size_t)t * a.kv_heads + u) * a.dim + i] = qv;
+        a.kn[((size_t)t * a.kv_heads + u) * a.dim + i] = kv;
+        qk = fmaf(qv, kv, qk);
+      }
+      if (a.head_decay) {
+        qk = mi::warp_sum(qk);
+        if (lane == 0) a.qk[(size_t)t * a.kv_heads + u] = qk;
       }
     } else {
       const int h = u - a.kv_heads;
       const float neg_rate = -expf(a.A_log[h]);
-      for (int i = lane; i < a.dim; i += 32) {
+      if (a.head_decay) {
+        if (lane == 0) a.g[(size_t)t * a.heads + h] = expf(neg_rate * softplus_f(mi::to_float(a.a[(size_t)t * a.lda + h]) + a.dt_bias[h]));
+      } else for (int i = lane; i < a.dim; i += 32) {
         const float z = mi::to_float(a.a[(size_t)t * a.lda + (size_t)h * a.dim + i]) + a.dt_bias[h * a.dim + i];
         a.g[((size_t)t * a.heads + h) * a.dim + i] = expf(neg_rate * softplus_f(z));
       }
@@ -349,13 +366,21 @@ __device__ __forceinline__ void copy4(float* dst, const float* src, bool take) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(d), "l"(src), "r"(bytes) : "memory");
 }
 
+// 16 bytes, both sides 16-byte aligned
+__device__ __forceinline__ void copy16(float* dst, const float* src, bool take) {
+  const unsigned d = (unsigned)__cvta_generic_to_shared(dst);
+  const int bytes = take ? 16 : 0;
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(bytes) : "memory");
+}
+
 constexpr int DELTA_THREADS = 128;
 constexpr int DELTA_CHUNK = 16;       // tokens whose vectors are in shared memory at a time
 
 template <typename T>
 struct DeltaArgs {
   float* raw;                            // [tokens, heads * vdim]: the values in, the read-outs before norm and gate out
-  const float* qn; const float* kn; const float* g; const float* beta;
+  const float* qn; const float* kn; const float* g; const float* beta; const float* qk;
+  int vec16;                             // rows of q, k, g and the values start on 16-byte boundaries and hold whole 16 bytes
   float* state; long long state_stride;  // [slot][heads][dim][vdim]
   const int* q_start; const int* q_len; const int* seq_slot;
   int heads, kv_heads, dim, vdim, R;
@@ -381,7 +406,10 @@ __host__ __device__ __forceinline__ int delta_segment_len(int n_new, int nseg) {
 // values, and dim more columns that start as the identity with zero values - they end as the stretch's map.  The carry
 // kernel chains the stretches; MODE 2 walks every stretch again from the state it really starts from and writes the
 // read-outs.
-template <typename T, int DK, int MODE>
+// Floats of one token in shared memory: the padded q, k (and g) vectors, the block's values, beta, g and q . k of the head.
+__host__ __device__ constexpr int delta_token_floats(int vec, int cols, bool head_decay) { return (head_decay ? 2 : 3) * vec + cols + 4; }
+
+template <typename T, int DK, int MODE, bool HEAD_DECAY>
 __global__ void __launch_bounds__(DELTA_THREADS)
 delta_recurrence_kernel(DeltaArgs<T> a) {
   extern __shared__ __align__(16) float sm[];
@@ -405,7 +433,8 @@ delta_recurrence_kernel(DeltaArgs<T> a) {
   const bool map_col = MODE == 1 && col >= vdim;             // a column of the stretch's map: starts as a unit vector, zero values
   const bool live = col < vdim + (MODE == 1 ? dim : 0);
   const int vec = R * LD;                                    // floats of one padded vector
-  const int tok_floats = 3 * vec + cols + 4;                 // q, k, g, the block's values, beta
+  const int tok_floats = delta_token_floats(vec, cols, HEAD_DECAY);
+  const int v_at = (HEAD_DECAY ? 2 : 3) * vec;               // the values, then the head's numbers
   mi::grid_dependency_sync();
   const size_t seg_at = ((size_t)(item * DELTA_SEGMENTS + seg) * a.heads + head) * dim;
   float* st = MODE == 0 ? a.state + (size_t)slot * a.state_stride + (size_t)head * dim * vdim : a.seg_state + seg_at * vdim;
@@ -422,22 +451,35 @@ delta_recurrence_kernel(DeltaArgs<T> a) {
   const int chunk_floats = DELTA_CHUNK * tok_floats;
   auto fetch = [&](int c0, float* buf) {
     const int n = min(DELTA_CHUNK, n_new - c0);
-    for (int idx = threadIdx.x; idx < n * R * DK; idx += DELTA_THREADS) {
-      const int tt = idx / (R * DK), i = idx % (R * DK);
+    auto rows = [&](auto width, auto copy) {
+      constexpr int W = decltype(width)::value;
+      const int per_vec = R * DK / W, per_val = cols / W;
+      for (int idx = threadIdx.x; idx < n * per_vec; idx += DELTA_THREADS) {
+        const int tt = idx / per_vec, i = (idx - tt * per_vec) * W;
+        const size_t t = (size_t)(row0 + c0 + tt);
+        float* base = buf + (size_t)tt * tok_floats + (i / DK) * LD + (i % DK);
+        const bool in = i < dim;
+        copy(base, a.qn + (t * a.kv_heads + kvh) * dim + (in ? i : 0), in);
+        copy(base + vec, a.kn + (t * a.kv_heads + kvh) * dim + (in ? i : 0), in);
+        if (!HEAD_DECAY) copy(base + 2 * vec, a.g + (t * a.heads + head) * dim + (in ? i : 0), in);
+      }
+      for (int idx = threadIdx.x; idx < n * per_val; idx += DELTA_THREADS) {
+        const int tt = idx / per_val, j = (idx - tt * per_val) * W;
+        const int c = blockIdx.z * cols + j;
+        copy(buf + (size_t)tt * tok_floats + v_at + j, a.raw + (size_t)(row0 + c0 + tt) * (a.heads * vdim) + head * vdim + (c < vdim ? c : 0), c < vdim);
+      }
+    };
+    if (a.vec16) rows(std::integral_constant<int, 4>(), [](float* d, const float* g, bool in) { copy16(d, g, in); });
+    else rows(std::integral_constant<int, 1>(), [](float* d, const float* g, bool in) { copy4(d, g, in); });
+    for (int tt = threadIdx.x; tt < n; tt += DELTA_THREADS) {
       const size_t t = (size_t)(row0 + c0 + tt);
-      float* base = buf + (size_t)tt * tok_floats + (i / DK) * LD + (i % DK);
-      const bool in = i < dim;
-      copy4(base, a.qn + (t * a.kv_heads + kvh) * dim + (in ? i : 0), in);
-      copy4(base + vec, a.kn + (t * a.kv_heads + kvh) * dim + (in ? i : 0), in);
-      copy4(base + 2 * vec, a.g + (t * a.heads + head) * dim + (in ? i : 0), in);
+      float* head_at = buf + (size_t)tt * tok_floats + v_at + cols;
+      copy4(head_at, a.beta + t * a.heads + head, true);
+      if (HEAD_DECAY) {
+        copy4(head_at + 1, a.g + t * a.heads + head, true);
+        copy4(head_at + 2, a.qk + t * a.kv_heads + kvh, true);
+      }
     }
-    for (int idx = threadIdx.x; idx < n * cols; idx += DELTA_THREADS) {
-      const int tt = idx / cols, j = idx % cols;
-      const int c = blockIdx.z * cols + j;
-      copy4(buf + (size_t)tt * tok_floats + 3 * vec + j, a.raw + (size_t)(row0 + c0 + tt) * (a.heads * vdim) + head * vdim + (c < vdim ? c : 0), c < vdim);
-    }
-    for (int tt = threadIdx.x; tt < n; tt += DELTA_THREADS)
-      copy4(buf + (size_t)tt * tok_floats + 3 * vec + cols, a.beta + (size_t)(row0 + c0 + tt) * a.heads + head, true);
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   if (n_new > 0) fetch(0, sm);
@@ -455,6 +497,36 @@ delta_recurrence_kernel(DeltaArgs<T> a) {
       const float* base = cur + (size_t)tt * tok_floats;
       const float4* qv = reinterpret_cast<const float4*>(base + r * LD);
       const float4* kv = reinterpret_cast<const float4*>(base + vec + r * LD);
+      if constexpr (HEAD_DECAY) {
+        const float* hd = base + v_at + cols;
+        const float beta = hd[0], g = hd[1], qk = hd[2];
+        float ks[4] = {0.f, 0.f, 0.f, 0.f}, os[4] = {0.f, 0.f, 0.f, 0.f};
+        float4 kr[DK / 4];
+#pragma unroll
+        for (int i = 0; i < DK / 4; ++i) {
+          const float4 k4 = kr[i] = kv[i];
+          ks[0] = fmaf(k4.x, S[4 * i], ks[0]); ks[1] = fmaf(k4.y, S[4 * i + 1], ks[1]);
+          ks[2] = fmaf(k4.z, S[4 * i + 2], ks[2]); ks[3] = fmaf(k4.w, S[4 * i + 3], ks[3]);
+          if (MODE != 1) {
+            const float4 q4 = qv[i];
+            os[0] = fmaf(q4.x, S[4 * i], os[0]); os[1] = fmaf(q4.y, S[4 * i + 1], os[1]);
+            os[2] = fmaf(q4.z, S[4 * i + 2], os[2]); os[3] = fmaf(q4.w, S[4 * i + 3], os[3]);
+          }
+        }
+        float kS = (ks[0] + ks[1]) + (ks[2] + ks[3]), qS = (os[0] + os[1]) + (os[2] + os[3]);
+        for (int o = R >> 1; o > 0; o >>= 1) {
+          kS += __shfl_xor_sync(0xffffffffu, kS, o);
+          if (MODE != 1) qS += __shfl_xor_sync(0xffffffffu, qS, o);
+        }
+        const float u = beta * fmaf(-g, kS, base[v_at + cl]);
+#pragma unroll
+        for (int i = 0; i < DK / 4; ++i) {
+          S[4 * i] = fmaf(kr[i].x, u, g * S[4 * i]); S[4 * i + 1] = fmaf(kr[i].y, u, g * S[4 * i + 1]);
+          S[4 * i + 2] = fmaf(kr[i].z, u, g * S[4 * i + 2]); S[4 * i + 3] = fmaf(kr[i].w, u, g * S[4 * i + 3]);
+        }
+        if (MODE != 1 && live && r == 0) a.raw[(size_t)(row0 + c0 + tt) * (a.heads * vdim) + head * vdim + col] = fmaf(qk, u, g * qS);
+        continue;
+      }
       const float4* gv = reinterpret_cast<const float4*>(base + 2 * vec + r * LD);
       float ks[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
@@ -466,7 +538,7 @@ delta_recurrence_kernel(DeltaArgs<T> a) {
       }
       float kS = (ks[0] + ks[1]) + (ks[2] + ks[3]);
       for (int o = R >> 1; o > 0; o >>= 1) kS += __shfl_xor_sync(0xffffffffu, kS, o);
-      const float u = base[3 * vec + cols] * (base[3 * vec + cl] - kS);
+      const float u = base[v_at + cols] * (base[v_at + cl] - kS);
       float os[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int i = 0; i < DK / 4; ++i) {
@@ -550,7 +622,7 @@ delta_carry_kernel(float* __restrict__ seg_state, const float* __restrict__ seg_
 template <typename T>
 __global__ void __launch_bounds__(128)
 delta_output_kernel(T* __restrict__ out, int ldo, const float* __restrict__ raw, const T* __restrict__ gate, int ldg,
-                    const float* __restrict__ norm_w, int heads, int vdim, float eps) {
+                    const float* __restrict__ norm_w, int heads, int vdim, float eps, int gate_silu) {
   mi::grid_dependency_sync();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int t = blockIdx.x;
@@ -562,7 +634,7 @@ delta_output_kernel(T* __restrict__ out, int ldo, const float* __restrict__ raw,
     const float rstd = 1.f / sqrtf(ss / (float)vdim + eps);
     for (int j = lane; j < vdim; j += 32) {
       const float gl = mi::to_float(gate[(size_t)t * ldg + h * vdim + j]);
-      out[(size_t)t * ldo + h * vdim + j] = mi::from_float<T>(o[j] * rstd * norm_w[j] * sigmoid_f(gl));
+      out[(size_t)t * ldo + h * vdim + j] = mi::from_float<T>(o[j] * rstd * norm_w[j] * (gate_silu ? silu_f(gl) : sigmoid_f(gl)));
     }
   }
 }
@@ -637,9 +709,9 @@ MI_API int mi_selective_scan(void* y, int ldy, const void* u, int ldu, const voi
   return 0;
 }
 
-// scratch: float32, tokens * (2 * kv_heads * dim + heads * dim + heads + heads * vdim) values (mi_gated_delta_scratch_floats)
-MI_API long long mi_gated_delta_scratch_floats(int T, int heads, int kv_heads, int dim, int vdim) {
-  return (long long)T * ((long long)2 * kv_heads * dim + (long long)heads * dim + heads + (long long)heads * vdim);
+// scratch: float32 - unit q and k, decays, q . k, beta, values / read-outs, each starting on a 16-byte boundary
+MI_API long long mi_gated_delta_scratch_floats(int T, int heads, int kv_heads, int dim, int vdim, int head_decay) {
+  return (long long)T * ((long long)2 * kv_heads * dim + (long long)heads * (head_decay ? 1 : dim) + kv_heads + heads + (long long)heads * vdim) + 5 * 4;
 }
 
 MI_API int mi_gated_delta_segments() { return DELTA_SEGMENTS; }
@@ -661,7 +733,8 @@ MI_API int mi_gated_delta(void* out, int ldo, const void* q, const void* k, int 
                           const void* b_in, int ldb, const void* gate, int ldg, int dtype, const float* dt_bias, const float* A_log,
                           const float* norm_w, float eps, float* state, long long state_stride, const int* q_start, const int* q_len,
                           const int* seq_slot, int T, int items, int heads, int kv_heads, int dim, int vdim, float* scratch,
-                          float* segments, cudaStream_t stream) {
+                          float* segments, int head_decay, int gate_silu, cudaStream_t stream) {
+  // head_decay: a_in [T, heads] and dt_bias [heads], one decay a head, instead of [T, heads * dim] and [heads * dim]
   // segments: null, or items * DELTA_SEGMENTS * heads * dim * (vdim + dim) floats of scratch - then the items' tokens run
   // in stretches side by side (bfloat16 only: the sums then depend on where a portion starts; dim up to 256)
   MI_REQUIRE(segments == nullptr || (dtype == MI_BF16 && dim <= 256 && items * DELTA_SEGMENTS <= 65535),
@@ -680,40 +753,45 @@ MI_API int mi_gated_delta(void* out, int ldo, const void* q, const void* k, int 
   }
   MI_REQUIRE(R <= 32, "gated_delta: dim=%d is more than a block's threads can keep", dim);
   const int cols = DELTA_THREADS / R;
-  const int tok_floats = 3 * R * (DK + 4) + cols + 4;
+  const int tok_floats = delta_token_floats(R * (DK + 4), cols, head_decay != 0);
   const size_t smem = (size_t)2 * DELTA_CHUNK * tok_floats * sizeof(float);
   MI_REQUIRE(smem <= 200 * 1024, "gated_delta: a chunk's vectors (%zu bytes) do not fit shared memory", smem);
+  auto up4 = [](size_t n) { return (n + 3) / 4 * 4; };
   float* qn = scratch;
-  float* kn = qn + (size_t)T * kv_heads * dim;
-  float* g = kn + (size_t)T * kv_heads * dim;
-  float* beta = g + (size_t)T * heads * dim;
-  float* raw = beta + (((size_t)T * heads + 3) / 4) * 4;
+  float* kn = qn + up4((size_t)T * kv_heads * dim);
+  float* g = kn + up4((size_t)T * kv_heads * dim);
+  float* qk = g + up4((size_t)T * heads * (head_decay ? 1 : dim));
+  float* beta = qk + up4((size_t)T * kv_heads);
+  float* raw = beta + up4((size_t)T * heads);
   dim3 pgrid(T, (heads + kv_heads + 3) / 4 > 16 ? 16 : (heads + kv_heads + 3) / 4);
   dim3 ogrid(T, (heads + 3) / 4 > 16 ? 16 : (heads + 3) / 4);
   dim3 rgrid(heads, items, (vdim + cols - 1) / cols);
 #define MI_DELTA(TT, DKV)                                                                                         \
+  do { if (head_decay) MI_DELTA_FORM(TT, DKV, true); else MI_DELTA_FORM(TT, DKV, false); } while (0)
+#define MI_DELTA_FORM(TT, DKV, HD)                                                                                \
   do {                                                                                                            \
     DeltaArgs<TT> d;                                                                                              \
-    d.raw = raw; d.qn = qn; d.kn = kn; d.g = g; d.beta = beta;                                                    \
+    d.raw = raw; d.qn = qn; d.kn = kn; d.g = g; d.beta = beta; d.qk = qk;                                         \
+    d.vec16 = dim % 4 == 0 && vdim % 4 == 0 && cols % 4 == 0;                                                     \
     d.state = state; d.state_stride = state_stride; d.q_start = q_start; d.q_len = q_len; d.seq_slot = seq_slot;  \
     d.heads = heads; d.kv_heads = kv_heads; d.dim = dim; d.vdim = vdim; d.R = R;                                  \
     d.seg_state = segments; d.seg_map = segments ? segments + (size_t)items * DELTA_SEGMENTS * heads * dim * vdim : nullptr; \
     if (!segments) {                                                                                              \
-      if (smem > 48 * 1024) cudaFuncSetAttribute(delta_recurrence_kernel<TT, DKV, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-      mi::launch(delta_recurrence_kernel<TT, DKV, 0>, rgrid, dim3(DELTA_THREADS), smem, stream, d);               \
+      if (smem > 48 * 1024) cudaFuncSetAttribute(delta_recurrence_kernel<TT, DKV, 0, HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+      mi::launch(delta_recurrence_kernel<TT, DKV, 0, HD>, rgrid, dim3(DELTA_THREADS), smem, stream, d);               \
     } else {                                                                                                      \
       if (smem > 48 * 1024) {                                                                                     \
-        cudaFuncSetAttribute(delta_recurrence_kernel<TT, DKV, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-        cudaFuncSetAttribute(delta_recurrence_kernel<TT, DKV, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        cudaFuncSetAttribute(delta_recurrence_kernel<TT, DKV, 1, HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        cudaFuncSetAttribute(delta_recurrence_kernel<TT, DKV, 2, HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
       }                                                                                                           \
       dim3 g1(heads, items * DELTA_SEGMENTS, (vdim + dim + cols - 1) / cols), g2(heads, items * DELTA_SEGMENTS, rgrid.z); \
       const int dimp = (dim + 31) / 32 * 32, TJ = 1024 / dimp;                                                    \
-      mi::launch(delta_recurrence_kernel<TT, DKV, 1>, g1, dim3(DELTA_THREADS), smem, stream, d);                  \
+      mi::launch(delta_recurrence_kernel<TT, DKV, 1, HD>, g1, dim3(DELTA_THREADS), smem, stream, d);                  \
       const size_t csmem = (size_t)dim * (TJ + (dim < CARRY_KT ? dim : CARRY_KT)) * sizeof(float);                \
       if (csmem > 48 * 1024) cudaFuncSetAttribute(delta_carry_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)csmem); \
       mi::launch(delta_carry_kernel, dim3(heads, items, (vdim + TJ - 1) / TJ), dim3(dimp * TJ), csmem, stream,    \
                  d.seg_state, (const float*)d.seg_map, state, state_stride, q_len, seq_slot, heads, dim, vdim, dimp, TJ); \
-      mi::launch(delta_recurrence_kernel<TT, DKV, 2>, g2, dim3(DELTA_THREADS), smem, stream, d);                  \
+      mi::launch(delta_recurrence_kernel<TT, DKV, 2, HD>, g2, dim3(DELTA_THREADS), smem, stream, d);                  \
     }                                                                                                             \
   } while (0)
 #define MI_DELTA_ALL(TT)                                                                                          \
@@ -721,19 +799,21 @@ MI_API int mi_gated_delta(void* out, int ldo, const void* q, const void* k, int 
     DeltaPrepArgs<TT> p;                                                                                          \
     p.q = (const TT*)q; p.k = (const TT*)k; p.ldqk = ldqk; p.a = (const TT*)a_in; p.lda = lda; p.b = (const TT*)b_in; p.ldb = ldb; \
     p.dt_bias = dt_bias; p.A_log = A_log; p.qn = qn; p.kn = kn; p.g = g; p.beta = beta; p.T_ = T; p.heads = heads;  \
+    p.qk = qk; p.head_decay = head_decay;                                                                         \
     p.kv_heads = kv_heads; p.dim = dim; p.v = (const TT*)v; p.ldv = ldv; p.raw = raw; p.vdim = vdim;                  \
     mi::launch(delta_prepare_kernel<TT>, pgrid, dim3(128), 0, stream, p);                                         \
     if (DK == 16) MI_DELTA(TT, 16);                                                                               \
     else if (DK == 32) MI_DELTA(TT, 32);                                                                          \
     else if (DK == 64) MI_DELTA(TT, 64);                                                                          \
     else MI_DELTA(TT, 128);                                                                                       \
-    mi::launch(delta_output_kernel<TT>, ogrid, dim3(128), 0, stream, (TT*)out, ldo, (const float*)raw, (const TT*)gate, ldg, norm_w, heads, vdim, eps); \
+    mi::launch(delta_output_kernel<TT>, ogrid, dim3(128), 0, stream, (TT*)out, ldo, (const float*)raw, (const TT*)gate, ldg, norm_w, heads, vdim, eps, gate_silu); \
   } while (0)
   if (dtype == MI_BF16) MI_DELTA_ALL(__nv_bfloat16);
   else if (dtype == MI_F32) MI_DELTA_ALL(float);
   else return mi_fail("gated_delta: unknown dtype %d", dtype);
 #undef MI_DELTA_ALL
 #undef MI_DELTA
+#undef MI_DELTA_FORM
   MI_LAUNCH_OK("gated_delta");
   return 0;
 }

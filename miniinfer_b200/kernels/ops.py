@@ -495,12 +495,13 @@ def _cols(t: torch.Tensor, what: str):
 
 
 def linear_batched(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, softplus: bool = False,
-                   row_gate: Optional[torch.Tensor] = None) -> None:
+                   row_gate: Optional[torch.Tensor] = None, value_gate: Optional[torch.Tensor] = None) -> None:
   """out[:, b, :] = x[:, b, :] @ w[b]^T for ``x [M, batch, K]``, ``w [batch, N, K]``, ``out [M, batch, N]`` - views whose
   strides may be anything as long as the last axis is contiguous (the heads of a token's row, a column range of a
-  row); float32 sums, k ascending.  bfloat16 with more than 16 rows and nothing behind the product: one strided batched library product.
+  row); float32 sums, k ascending.  bfloat16 with more than 16 rows and nothing but a gate a value behind the product: one
+  strided batched library product, the gate in a kernel behind it.
   ``bias [N]`` float32 is added, ``softplus`` applied, and with ``row_gate [M, >= batch]``
-  (one logit per row and batch) the result is multiplied with its sigmoid."""
+  (one logit per row and batch) or ``value_gate [M, batch * N]`` (one per output value) the result is multiplied with its sigmoid."""
   lib = common_lib()
   M, B, K = x.shape
   N = w.shape[1]
@@ -516,10 +517,15 @@ def linear_batched(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, bias: Op
     if row_gate.dim() != 2 or row_gate.shape[0] != M or row_gate.shape[1] < B or row_gate.stride(1) != 1 or row_gate.dtype != x.dtype:
       raise KernelError("linear_batched: the row gate must hold a logit per row and batch, in the operands' dtype")
     gate_stride = row_gate.stride(0)
+  if value_gate is not None:
+    if (row_gate is not None or value_gate.dim() != 2 or value_gate.shape != (M, B * N) or value_gate.stride(1) != 1 or value_gate.dtype != x.dtype
+        or not value_gate.is_cuda):
+      raise KernelError("linear_batched: the value gate must hold a logit per output value, in the operands' dtype, and goes without a row gate")
+    gate_stride = value_gate.stride(0)
   few = M <= 16 and x.dtype == torch.bfloat16
   aligned = K % 8 == 0 and all(t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0 and t.stride(1) % 8 == 0 for t in (x, w, out))
   if (x.dtype == torch.bfloat16 and not few and out.dtype == torch.bfloat16 and bias is None and row_gate is None and not softplus
-      and B > 1 and w.stride(1) == K and aligned):
+      and B > 1 and w.stride(1) == K and aligned and (value_gate is None or out.stride(1) == N)):
     # many rows and nothing behind the product: the library's, all parts in one call (torch's while a graph is recorded)
     if not _capturing:
       _check(lib, lib.mi_gemm_cublas_bf16_batched(
@@ -528,12 +534,16 @@ def linear_batched(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, bias: Op
         kernels=0)
     else:
       torch.bmm(x.transpose(0, 1), w.transpose(1, 2), out=out.transpose(0, 1))
+    if value_gate is not None:
+      _check(lib, lib.mi_sigmoid_gate_bf16(ctypes.c_void_p(out.data_ptr()), ctypes.c_longlong(out.stride(0)), ctypes.c_void_p(value_gate.data_ptr()),
+                                           ctypes.c_longlong(gate_stride), M, B * N, _stream()))
     return
   _check(lib, (lib.mi_gemm_batched_few_rows if few else lib.mi_gemm_batched)(
     ctypes.c_void_p(out.data_ptr()), _dt(out), ctypes.c_void_p(x.data_ptr()), ctypes.c_void_p(w.data_ptr()), _dt(x), B, M, N, K,
     int(x.stride(0)), ctypes.c_longlong(x.stride(1)), int(w.stride(1)), ctypes.c_longlong(w.stride(0)),
     int(out.stride(0)), ctypes.c_longlong(out.stride(1)), _ptr(bias, torch.float32) if bias is not None else _ptr(None),
-    int(bool(softplus)), ctypes.c_void_p(row_gate.data_ptr()) if row_gate is not None else _ptr(None), gate_stride, _stream()))
+    int(bool(softplus)), ctypes.c_void_p(row_gate.data_ptr()) if row_gate is not None else _ptr(None), gate_stride,
+    ctypes.c_void_p(value_gate.data_ptr()) if value_gate is not None else _ptr(None), _stream()))
 
 
 def linear_parts(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor) -> None:
@@ -631,20 +641,23 @@ def selective_scan(y: torch.Tensor, u: torch.Tensor, dt_in: torch.Tensor, bc: to
 
 def gated_delta(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch.Tensor, b: torch.Tensor, gate: torch.Tensor,
                 dt_bias: torch.Tensor, A_log: torch.Tensor, norm_w: torch.Tensor, eps: float, state: torch.Tensor, ctx,
-                heads: int, kv_heads: int, dim: int, vdim: int, workspace=None) -> None:
+                heads: int, kv_heads: int, dim: int, vdim: int, workspace=None, gate_silu: bool = False) -> None:
   """The gated delta rule over each item's new tokens, from and to the per-request state ``[slots, >= heads * dim * vdim]``
   float32.  ``q``, ``k`` ``[T, kv_heads * dim]`` (convolved and activated; made unit vectors here, q also times dim^-1/2),
   ``v [T, heads * vdim]``, ``a [T, heads * dim]`` (decay input: g = exp(-exp(A_log_h) softplus(a + dt_bias))), ``b [T, heads]``
   (beta = sigmoid(b)), ``gate [T, heads * vdim]``; per head ``S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q``;
-  ``out = o / rms(o) * norm_w * sigmoid(gate)``.  All operands may be column ranges of wider rows.  Three launches: what
+  ``out = o / rms(o) * norm_w * sigmoid(gate)``, or ``silu(gate)`` with ``gate_silu``.  ``a [T, heads]`` with ``dt_bias [heads]`` is
+  one decay a head.  All operands may be column ranges of wider rows.  Three launches: what
   does not depend on the state for all tokens at once, the recurrence, the read-outs' norm and gate; float32 scratch
   between them from ``workspace`` (a ``Workspace``; made here if absent).  A bfloat16 step of long prompt portions walks
   each request's tokens in stretches side by side (``csrc/recurrent.cu``); a float32 step walks them in order, so that its
   sums do not depend on how a request was cut."""
   lib = common_lib()
   T = v.shape[0]
-  if (q.shape != (T, kv_heads * dim) or k.shape != q.shape or v.shape != (T, heads * vdim) or a.shape != (T, heads * dim) or b.shape != (T, heads)
-      or gate.shape != v.shape or out.shape != v.shape or dt_bias.shape != (heads * dim,) or A_log.shape != (heads,) or norm_w.shape != (vdim,)):
+  head_decay = dt_bias.shape == (heads,)
+  decays = heads if head_decay else heads * dim
+  if (q.shape != (T, kv_heads * dim) or k.shape != q.shape or v.shape != (T, heads * vdim) or a.shape != (T, decays) or b.shape != (T, heads)
+      or gate.shape != v.shape or out.shape != v.shape or dt_bias.shape != (decays,) or A_log.shape != (heads,) or norm_w.shape != (vdim,)):
     raise KernelError("gated_delta: shapes do not match")
   if len({t.dtype for t in (out, q, k, v, a, b, gate)}) != 1:
     raise KernelError("gated_delta: the activations differ in dtype")
@@ -654,7 +667,7 @@ def gated_delta(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Te
   if ldq != ldk:
     raise KernelError("gated_delta: q and k must be column ranges of rows of one width")
   lib.mi_gated_delta_scratch_floats.restype = ctypes.c_longlong
-  n = int(lib.mi_gated_delta_scratch_floats(T, heads, kv_heads, dim, vdim)) + 8
+  n = int(lib.mi_gated_delta_scratch_floats(T, heads, kv_heads, dim, vdim, int(head_decay))) + 8
   scratch = workspace.buffer("gated_delta_scratch", (n,), torch.float32) if workspace is not None else \
     torch.empty(n, dtype=torch.float32, device=v.device)
   # long prompt portions in bfloat16: each request's tokens in up to 16 stretches side by side (five launches instead of three)
@@ -671,7 +684,7 @@ def gated_delta(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Te
                                  ctypes.c_void_p(state.data_ptr()), ctypes.c_longlong(state.stride(0)), _ptr(ctx.q_start, torch.int32),
                                  _ptr(ctx.q_len, torch.int32), _ptr(ctx.seq_slot, torch.int32), T, ctx.num_items, heads, kv_heads, dim, vdim,
                                  _ptr(scratch, torch.float32), _ptr(segments, torch.float32) if segments is not None else _ptr(None),
-                                 _stream()), kernels=launches)
+                                 int(head_decay), int(gate_silu), _stream()), kernels=launches)
 
 
 LINEAR_SEGMENTED_MAX_ITEMS = 8     # steps of at most this many requests run long bfloat16 portions in stretches side by side
@@ -971,16 +984,19 @@ def scaled_pair_sum(out: torch.Tensor, a: torch.Tensor, b: torch.Tensor, scale_a
 
 
 def latent_down(down: torch.Tensor, q_off: int, kv_off: int, q_rank: int, kv_rank: int, rot_dim: int, q_weight: torch.Tensor,
-                kv_weight: torch.Tensor, eps: float, cq_out: torch.Tensor, rope: torch.Tensor, positions: torch.Tensor, interleaved: bool,
+                kv_weight: Optional[torch.Tensor], eps: float, cq_out: torch.Tensor, rope: torch.Tensor, positions: torch.Tensor, interleaved: bool,
                 slot_mapping: Optional[torch.Tensor], kv_layer: Optional[torch.Tensor]) -> None:
   """From the fused down-projection rows of a latent attention: the RMS-normed query latent (``q_rank`` values at ``q_off``)
   into ``cq_out [T, q_rank]``; the RMS-normed key/value latent (``kv_rank`` values at ``kv_off``) and the rotated shared key
-  part (``rot_dim`` values behind it) into the layer's pages: key row ``[c | k_rot | 0]``, value row ``[c | 0]``."""
+  part (``rot_dim`` values behind it) into the layer's pages: key row ``[c | k_rot | 0]``, value row ``[c | 0]``.  ``kv_weight`` None:
+  the rows hold a query latent only, and nothing is stored."""
   lib = common_lib()
   T = down.shape[0]
-  if max(q_off + q_rank, kv_off + kv_rank + rot_dim) > down.shape[1] or cq_out.shape != (T, q_rank) or cq_out.dtype != down.dtype:
+  if kv_weight is None and kv_layer is not None:
+    raise KernelError("latent_down: rows without a key/value latent cannot be stored")
+  if max(q_off + q_rank, kv_off + kv_rank + rot_dim if kv_weight is not None else 0) > down.shape[1] or cq_out.shape != (T, q_rank) or cq_out.dtype != down.dtype:
     raise KernelError("latent_down: the latents do not fit the projection rows")
-  if rope.shape[1] != rot_dim or q_weight.shape != (q_rank,) or kv_weight.shape != (kv_rank,):
+  if rope.shape[1] != rot_dim or q_weight.shape != (q_rank,) or (kv_weight is not None and kv_weight.shape != (kv_rank,)):
     raise KernelError("latent_down: weights or rotation table do not match")
   hdp, page_size = kv_rank + rot_dim, 0
   if kv_layer is not None:
@@ -989,7 +1005,7 @@ def latent_down(down: torch.Tensor, q_off: int, kv_off: int, q_rank: int, kv_ran
     page_size, hdp = kv_layer.shape[3], kv_layer.shape[4]
   none = _ptr(None)
   _check(lib, lib.mi_latent_down(_ptr(down), _dt(down), down.shape[1], q_off, kv_off, T, q_rank, kv_rank, rot_dim, hdp,
-                                 _ptr(q_weight, torch.float32), _ptr(kv_weight, torch.float32), ctypes.c_float(eps), _ptr(cq_out),
+                                 _ptr(q_weight, torch.float32), _ptr(kv_weight, torch.float32) if kv_weight is not None else none, ctypes.c_float(eps), _ptr(cq_out),
                                  _ptr(rope, torch.float32), _ptr(positions, torch.int32), int(bool(interleaved)),
                                  _ptr(slot_mapping, torch.int32) if (slot_mapping is not None and kv_layer is not None) else none,
                                  _ptr(kv_layer) if kv_layer is not None else none, page_size, _stream()))
@@ -1022,7 +1038,7 @@ def moe_rows(num_pairs: int, num_experts: int, tile: int) -> int:
   return -(-(num_pairs + num_experts * (tile - 1)) // tile) * tile
 
 
-GLU_KINDS = {"silu": 0, "clamped": 1}      # the gated activations of common.cuh (MiGlu)
+GLU_KINDS = {"silu": 0, "clamped": 1, "gelu_tanh": 2}      # the gated activations of common.cuh (MiGlu)
 
 
 def _glu(kind: str, limit: float):
@@ -1044,7 +1060,8 @@ def routed_experts(out: torch.Tensor, x: torch.Tensor, router: torch.Tensor, cor
 
   ``weights="softmax_chosen"``: the ``top`` largest logits are chosen (``correction`` may be None) and the weights are the
   softmax over the chosen logits alone.  ``glu``/``limit``: the experts' gated activation (``silu``, or ``clamped`` with its
-  limit: ``g' = min(g, L)``, ``u' = clamp(u, -L, L)``, ``g' sigmoid(1.702 g') (u' + 1)``).  ``shared [T, H]``: the output of an
+  limit: ``g' = min(g, L)``, ``u' = clamp(u, -L, L)``, ``g' sigmoid(1.702 g') (u' + 1)``, or ``gelu_tanh``: ``g / 2 (1 + tanh(sqrt(2 / pi)
+  (g + 0.044715 g^3))) u``).  ``shared [T, H]``: the output of an
   expert that every token runs through, added to the sum; with ``shared_gated`` the router has one row more than there are
   experts, and the shared rows are multiplied with the sigmoid of that row's logit, one number a token.
 
@@ -1178,10 +1195,11 @@ def glu_mul(out: torch.Tensor, gate_up: torch.Tensor, glu: str = "silu", limit: 
   _check(lib, lib.mi_glu_mul(_ptr(out), _ptr(gate_up), _dt(out), T, I, kind, lim, _stream()))
 
 
-def linear_glu(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, workspace, glu: str = "silu", limit: float = 0.0) -> None:
+def linear_glu(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, workspace, glu: str = "silu", limit: float = 0.0,
+               force_stream: bool = False) -> None:
   """out[M, I] = act(x @ w[:I]^T) * (x @ w[I:]^T): the gate-and-up product of a gated feed-forward with the activation
   ``glu``.  ``silu`` is ``linear_swiglu``; the others take the few-row mma.sync kernel with the activation in its epilogue up to 16
-  rows, the tcgen05 kernel with the activation in its epilogue from the same number of rows on as SwiGLU, and the product
+  rows (``gelu_tanh`` over a large matrix the tcgen05 streaming kernel), the tcgen05 kernel with the activation in its epilogue from the same number of rows on as SwiGLU, and the product
   followed by the activation kernel between."""
   if glu == "silu":
     linear_swiglu(out, x, w, workspace)
@@ -1193,6 +1211,12 @@ def linear_glu(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, workspace, g
   if M == 0:
     return
   kind, lim = _glu(glu, limit)
+  if glu == "gelu_tanh" and x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and _streams(M, 2 * I, K, False, force_stream):
+    lib = common_lib()
+    parts, counters, status = _stream_workspace(lib, x.device)
+    _check(lib, lib.mi_gemm_stream_tc_geglu_bf16(_ptr(out), _ptr(x), _ptr(w), M, I, K, I, _ptr(parts, torch.float32), _ptr(counters, torch.int32),
+                                                 counters.numel(), parts.shape[0], _ptr(status, torch.int32), _stream()))
+    return
   if (x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and M <= SKINNY_BEST_M and K % 8 == 0 and x.is_contiguous() and w.is_contiguous()
       and out.is_contiguous()):
     lib = common_lib()      # few rows: the weight-streaming product with the activation in its epilogue

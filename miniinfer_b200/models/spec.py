@@ -14,7 +14,7 @@ from __future__ import annotations
 from dataclasses import dataclass, field
 from typing import Dict, List, Optional
 
-from ..cache.specs import CacheSpec
+from ..cache.specs import CacheSpec, shared_need
 from ..config.model_config import ModelConfig
 from ..parts.base import Block, Embedding, Head, Norm, Part, PositionEncoding
 
@@ -54,8 +54,12 @@ class ModelSpec:
           raise ValueError(f"run list entry {i} reads the cache of entry {run.cache_of}, which has none of its own")
         a = self.blocks[run.block].mixer_part()
         b = self.blocks[self.run_list[run.cache_of].block].mixer_part()
-        if a is None or b is None or a.cache_spec() != b.cache_spec():
-          raise ValueError(f"run list entry {i} and entry {run.cache_of} differ in what they keep in the cache")
+        try:
+          if a is None or b is None:
+            raise ValueError("a block without a mixer")
+          shared_need([b.cache_spec(), a.cache_spec()])
+        except ValueError as e:
+          raise ValueError(f"run list entry {i} and entry {run.cache_of} differ in what they keep in the cache: {e}") from None
 
   def all_parts(self) -> List[Part]:
     out: List[Part] = [self.embedding]
@@ -73,8 +77,14 @@ class ModelSpec:
     return out
 
   def cache_layer_specs(self) -> List[Optional[CacheSpec]]:
-    """The cache need of every run-list entry (None: it keeps nothing of its own)."""
-    specs: List[Optional[CacheSpec]] = []
+    """The cache need of every run-list entry (None: it keeps nothing of its own).  An entry whose cache later entries read
+    keeps what any of them can see."""
+    readers: Dict[int, List[CacheSpec]] = {}
     for run in self.run_list:
-      specs.append(None if run.cache_of is not None else self.blocks[run.block].cache_spec())
+      if run.cache_of is not None:
+        readers.setdefault(run.cache_of, []).append(self.blocks[run.block].cache_spec())
+    specs: List[Optional[CacheSpec]] = []
+    for i, run in enumerate(self.run_list):
+      own = None if run.cache_of is not None else self.blocks[run.block].cache_spec()
+      specs.append(shared_need([own] + readers[i]) if i in readers else own)
     return specs

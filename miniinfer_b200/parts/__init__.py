@@ -10,7 +10,7 @@ from .latent_attention import LatentAttentionMixer
 from .linear_attention import LinearAttentionMixer
 from .mixer import AttentionMixer
 from .norm import LayerNorm, RMSNorm
-from .position import BandScaledRotaryEncoding, RotaryEncoding, ScaledRotaryEncoding
+from .position import BandScaledRotaryEncoding, LinearScaledRotaryEncoding, RotaryEncoding, ScaledRotaryEncoding
 from .recurrent import GatedDeltaMixer, MinGruMixer, RglruMixer, SelectiveScanMixer
 from .side_by_side import SideBySideMixer
 from .registry import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, POSITION_ENCODINGS, make, register_block,
@@ -35,6 +35,7 @@ register_norm("depth_average")(DepthAverageNorm)
 register_position_encoding("rotary")(RotaryEncoding)
 register_position_encoding("scaled_rotary")(ScaledRotaryEncoding)
 register_position_encoding("band_scaled_rotary")(BandScaledRotaryEncoding)
+register_position_encoding("linear_scaled_rotary")(LinearScaledRotaryEncoding)
 register_block("pre_norm")(PreNormBlock)
 register_block("parallel")(ParallelBlock)
 register_block("hyper_connection")(HyperConnectionBlock)

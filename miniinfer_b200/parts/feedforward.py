@@ -1,4 +1,4 @@
-"""Dense SwiGLU feed-forward: ``down(silu(gate(x)) * up(x))`` with gate and up in one matrix
+"""Dense gated feed-forward: ``down(silu(gate(x)) * up(x))``, or another gated activation, with gate and up in one matrix
 (miniinfer/models/fused_qwen3.py:111-138; order gate, up: miniinfer/loader/weight.py:87-93).
 """
 
@@ -14,7 +14,9 @@ from .base import FeedForward, ParamSpec, Piece, whole
 
 class SwiGLUFeedForward(FeedForward):
   """``activation``: ``silu``, or ``clamped`` with its ``limit``: ``g = min(gate x, limit)``, ``u = clamp(up x, -limit, limit)``,
-  ``g * sigmoid(1.702 g) * (u + 1)`` in place of ``silu(gate x) * up x``.  ``tensors``: the file names of the gate, up and down matrices after ``<name>.`` (default: ``gate_proj.weight``,
+  ``g * sigmoid(1.702 g) * (u + 1)`` in place of ``silu(gate x) * up x``, or ``gelu_tanh``: ``gelu_tanh(gate x) * up x`` with
+  ``gelu_tanh(z) = z / 2 (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))``.  ``tensors``: the file names of the gate, up and down
+  matrices after ``<name>.`` (default: ``gate_proj.weight``,
   ``up_proj.weight``, ``down_proj.weight``, with ``gate_up_proj.weight`` accepted for the fused pair)."""
 
   def __init__(self, name: str, hidden_size: int, intermediate_size: int, tensors: Optional[Tuple[str, str, str]] = None,

@@ -13,7 +13,11 @@ values and ``vdim`` value values, a query latent of ``q_rank`` and a key/value l
     is applied to the query instead, once per token, and attention runs over ONE key/value head whose key row is
     ``[c | k_rot]`` and whose value row is ``c``: ``H`` query heads of ``kv_rank + rot_dim`` values on it (sink in the softmax's
     denominator if ``sinks``), each giving ``sum_j p_j c_j``, which ``W_uv`` of the head then takes to ``vdim`` values;
-  * ``gated``: head h's output is multiplied by ``sigmoid((W_g h)_h)``, one gate a head; then the output projection.
+  * ``gated``: head h's output is multiplied by ``sigmoid((W_g h)_h)``, one gate a head, or - ``gate_per_head`` off - the
+    concatenated outputs element by element by ``sigmoid(W_g h)``; then the output projection;
+  * ``window``: token ``i`` sees token ``j`` of its request if ``0 <= i - j < window`` (None: every earlier token);
+  * ``keeps_latents`` off: there is no ``W_dkv``; the layer reads the latents and rotated key parts another layer has cached
+    (its entry of the run list names that layer's), with queries, up-projections and window of its own.
 
 The cache keeps rows of ``kv_rank + rot_dim`` values rounded up to a multiple of 16, zero-filled (rows of more than 256 values
 take the attention kernel without tensor cores).  The two per-head
@@ -35,9 +39,10 @@ from .mixer import AttentionMixer
 class LatentAttentionMixer(AttentionMixer):
   def __init__(self, name: str, hidden_size: int, num_heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int, kv_rank: int,
                scale: float, norm_eps: float, rotary: PositionEncoding, rotary_interleaved: bool = False, sinks: bool = True,
-               gated: bool = True, tensors: Optional[Dict[str, str]] = None):
+               gated: bool = True, tensors: Optional[Dict[str, str]] = None, gate_per_head: bool = True, window: Optional[int] = None,
+               keeps_latents: bool = True):
     cache_hd = -(-(kv_rank + rot_dim) // 16) * 16
-    super().__init__(name, hidden_size, num_heads, 1, cache_hd, scale, norm_eps, rotary, None)
+    super().__init__(name, hidden_size, num_heads, 1, cache_hd, scale, norm_eps, rotary, window)
     for what, v in (("dim", dim), ("rot_dim", rot_dim), ("vdim", vdim), ("q_rank", q_rank), ("kv_rank", kv_rank)):
       if v <= 0:
         raise ValueError(f"{name}: {what} must be positive, got {v}")
@@ -47,32 +52,37 @@ class LatentAttentionMixer(AttentionMixer):
     self.cache_head_dim = cache_hd
     self.rotary_interleaved = bool(rotary_interleaved)
     self.sinks, self.gated = bool(sinks), bool(gated)
+    self.gate_per_head, self.keeps_latents = bool(gate_per_head), bool(keeps_latents)
     t = {"dq": "dq", "dq_norm": "dq.norm", "uq": "uq", "dkv": "dkv", "dkv_norm": "dkv.norm", "uk": "uk", "uv": "uv", "g": "g",
          "o": "o", "sink": "sink"}
     t.update(tensors or {})
     self.tensors = t
     self.q_off, self.kv_off = 0, q_rank
-    self.g_off = q_rank + kv_rank + rot_dim
-    self.down_width = self.g_off + (num_heads if gated else 0)
+    self.g_off = q_rank + (kv_rank + rot_dim if keeps_latents else 0)
+    self.gate_width = 0 if not gated else (num_heads if gate_per_head else num_heads * vdim)
+    self.down_width = self.g_off + self.gate_width
 
   def cache_spec(self) -> Optional[CacheSpec]:
-    return PagedKVSpec(1, self.cache_head_dim, None)
+    return PagedKVSpec(1, self.cache_head_dim, self.window)
 
   def param_specs(self) -> Dict[str, ParamSpec]:
     W, H, D, R, Dv, Q, C, n, t = (self.hidden_size, self.num_heads, self.dim, self.rot_dim, self.vdim, self.q_rank, self.kv_rank,
                                   self.name, self.tensors)
-    pieces = [Piece(f"{n}.{t['dq']}", self.q_off, (Q, W)), Piece(f"{n}.{t['dkv']}", self.kv_off, (C + R, W))]
+    pieces = [Piece(f"{n}.{t['dq']}", self.q_off, (Q, W))]
+    if self.keeps_latents:
+      pieces.append(Piece(f"{n}.{t['dkv']}", self.kv_off, (C + R, W)))
     if self.gated:
-      pieces.append(Piece(f"{n}.{t['g']}", self.g_off, (H, W)))
+      pieces.append(Piece(f"{n}.{t['g']}", self.g_off, (self.gate_width, W)))
     specs = {
       "down": ParamSpec((self.down_width, W), "matrix", [pieces]),
       "dq_norm": ParamSpec((Q,), "vector", [whole(f"{n}.{t['dq_norm']}", (Q,))], init="ones_noise"),
-      "dkv_norm": ParamSpec((C,), "vector", [whole(f"{n}.{t['dkv_norm']}", (C,))], init="ones_noise"),
       "uq": ParamSpec((H * (D + R), Q), "matrix", [whole(f"{n}.{t['uq']}", (H * (D + R), Q))]),
       "uk": ParamSpec((H * D, C), "matrix", [whole(f"{n}.{t['uk']}", (H * D, C))]),
       "uv": ParamSpec((H * Dv, C), "matrix", [whole(f"{n}.{t['uv']}", (H * Dv, C))]),
       "o": ParamSpec((W, H * Dv), "matrix", [whole(f"{n}.{t['o']}", (W, H * Dv))]),
     }
+    if self.keeps_latents:
+      specs["dkv_norm"] = ParamSpec((C,), "vector", [whole(f"{n}.{t['dkv_norm']}", (C,))], init="ones_noise")
     if self.sinks:
       specs["sink"] = ParamSpec((H,), "vector", [whole(f"{n}.{t['sink']}", (H,))])
     return specs
@@ -98,12 +108,14 @@ class LatentAttentionMixer(AttentionMixer):
     H, D, R, Dv, Q, C, hdp = self.num_heads, self.dim, self.rot_dim, self.vdim, self.q_rank, self.kv_rank, self.cache_head_dim
     if cache.kind != "paged":
       raise RuntimeError(f"{self.name}: attention needs a paged cache, got {cache.kind!r}")
+    if cache.writes and not self.keeps_latents:
+      raise RuntimeError(f"{self.name}: a layer without latents of its own must read another layer's cache")
     table = self.position.rotary_table()
     down = ctx.ws.buffer("latent_down", (T, self.down_width), ctx.dtype)
     ops.linear(down, x, self.down)
     cq = ctx.ws.buffer("latent_cq", (T, Q), ctx.dtype)
-    ops.latent_down(down, self.q_off, self.kv_off, Q, C, R, self.dq_norm, self.dkv_norm, self.qk_norm_eps, cq, table, ctx.positions,
-                    self.rotary_interleaved, ctx.slot_mapping[cache.group] if cache.writes else None,
+    ops.latent_down(down, self.q_off, self.kv_off, Q, C, R, self.dq_norm, self.dkv_norm if self.keeps_latents else None,
+                    self.qk_norm_eps, cq, table, ctx.positions, self.rotary_interleaved, ctx.slot_mapping[cache.group] if cache.writes else None,
                     cache.tensor if cache.writes else None)
     q = ctx.ws.buffer("latent_q", (T, H * (D + R)), ctx.dtype)
     ops.linear(q, cq, self.uq)
@@ -111,11 +123,12 @@ class LatentAttentionMixer(AttentionMixer):
     ops.latent_query(q, q_heads, H, D, R, C, table, ctx.positions, self.rotary_interleaved)
     ops.linear_batched(q_heads.view(T, H, hdp)[:, :, :C], q.view(T, H, D + R)[:, :, :D], self.uk_t)
     attn = ctx.ws.buffer("attn_out", (T, H * C), ctx.dtype)
-    ops.attention(attn, q_heads, cache.tensor, ctx.block_tables[cache.group], self._batch(ctx), H, 1, hdp, self.scale, None,
+    ops.attention(attn, q_heads, cache.tensor, ctx.block_tables[cache.group], self._batch(ctx), H, 1, hdp, self.scale, self.window,
                   sink=self.sink if self.sinks else None, out_hd=C)
     heads = ctx.ws.buffer("latent_heads", (T, H * Dv), ctx.dtype)
-    ops.linear_batched(heads.view(T, H, Dv), attn.view(T, H, C), self.uv_heads,
-                       row_gate=down[:, self.g_off:self.g_off + H] if self.gated else None)
+    gate = down[:, self.g_off:self.g_off + self.gate_width] if self.gated else None
+    ops.linear_batched(heads.view(T, H, Dv), attn.view(T, H, C), self.uv_heads, row_gate=gate if self.gate_per_head else None,
+                       value_gate=gate if not self.gate_per_head else None)
     out = ctx.ws.buffer(self.out_buffer, (T, self.hidden_size), ctx.dtype)
     ops.linear(out, heads, self.o)
     return out

@@ -117,3 +117,19 @@ class BandScaledRotaryEncoding(RotaryEncoding):
   def build_table(self, positions: int) -> torch.Tensor:
     angles = torch.arange(positions, dtype=torch.float64)[:, None] * self.frequencies()[None, :]
     return torch.cat((angles.cos(), angles.sin()), dim=-1).float().contiguous()
+
+
+class LinearScaledRotaryEncoding(RotaryEncoding):
+  """Rotary angles of positions divided by a constant: ``f_i = theta^(-2i/dims) / factor``, every frequency alike.  Angles are
+  made in float64 and rounded once.  ``factor`` 1 is the plain table."""
+
+  def __init__(self, name: str, rotary_dim: int, theta: float, max_position_embeddings: int, factor: float = 1.0):
+    super().__init__(name, rotary_dim, theta, max_position_embeddings)
+    if not factor > 0:
+      raise ValueError(f"{name}: the factor must be positive, got {factor!r}")
+    self.factor = float(factor)
+
+  def build_table(self, positions: int) -> torch.Tensor:
+    f = self.theta ** (-2.0 * torch.arange(0, self.rotary_dim // 2, dtype=torch.float64) / self.rotary_dim) / self.factor
+    angles = torch.arange(positions, dtype=torch.float64)[:, None] * f[None, :]
+    return torch.cat((angles.cos(), angles.sin()), dim=-1).float().contiguous()

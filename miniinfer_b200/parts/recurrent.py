@@ -102,33 +102,44 @@ class GatedDeltaMixer(Mixer):
     per head ``S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q`` (the read-out sees the token's own write);
     ``o <- o / sqrt(mean(o^2) + eps) * norm * sigmoid(W_g2 (W_g1 h))``; out = ``W_o o``.
 
+  ``decay_rank`` None: one decay a head, ``g = exp(-exp(A_log_h) softplus(W_a h + dt_bias))`` with a row of ``W_a`` and a value of
+  ``dt_bias`` a head.  ``gate_rank`` None: the output gate's logits are ``W_g h``.  ``gate="silu"``: the gate is ``silu`` of its logits.
+
   Decays, gates of the recurrence, unit norms and the state are float32.  One fused product gives q, k, v, beta's logits and
-  the two low-rank inputs; one convolution runs over the q, k and v channels together.  File tensors (after ``<name>.``):
-  ``q``, ``q.conv``, ``k``, ``k.conv``, ``v``, ``v.conv``, ``b``, ``A_log``, ``norm``, ``a1``, ``a2``, ``dt_bias``, ``g1``, ``g2``, ``o``."""
+  the two low-rank inputs (or the decays' and the gate's logits themselves); one convolution runs over the q, k and v channels
+  together.  File tensors (after ``<name>.``):
+  ``q``, ``q.conv``, ``k``, ``k.conv``, ``v``, ``v.conv``, ``b``, ``A_log``, ``norm``, ``dt_bias``, ``o``; ``a1``, ``a2`` or ``a``; ``g1``, ``g2`` or ``g``."""
 
   def __init__(self, name: str, hidden_size: int, num_heads: int, num_kv_heads: int, dim: int, vdim: int, taps: int,
-               decay_rank: int, gate_rank: int, norm_eps: float, tensors: Optional[Dict[str, str]] = None):
+               decay_rank: Optional[int], gate_rank: Optional[int], norm_eps: float, tensors: Optional[Dict[str, str]] = None,
+               gate: str = "sigmoid"):
     super().__init__(name)
     if num_heads <= 0 or num_kv_heads <= 0 or num_heads % num_kv_heads:
       raise ValueError(f"{name}: heads={num_heads} must be a multiple of kv_heads={num_kv_heads}")
     for what, v in (("dim", dim), ("vdim", vdim), ("taps", taps), ("decay_rank", decay_rank), ("gate_rank", gate_rank)):
-      if v <= 0:
+      if v is not None and v <= 0:
         raise ValueError(f"{name}: {what} must be positive, got {v}")
+    if gate not in ("sigmoid", "silu"):
+      raise ValueError(f"{name}: gate must be 'sigmoid' or 'silu', got {gate!r}")
+    self.gate_silu = gate == "silu"
     self.hidden_size, self.num_heads, self.num_kv_heads, self.dim, self.vdim, self.taps = hidden_size, num_heads, num_kv_heads, dim, vdim, taps
     self.decay_rank, self.gate_rank, self.norm_eps = decay_rank, gate_rank, float(norm_eps)
-    t = {"q": "q", "k": "k", "v": "v", "b": "b", "a1": "a1", "a2": "a2", "g1": "g1", "g2": "g2", "o": "o", "A_log": "A_log",
+    t = {"q": "q", "k": "k", "v": "v", "b": "b", "a": "a", "g": "g", "a1": "a1", "a2": "a2", "g1": "g1", "g2": "g2", "o": "o", "A_log": "A_log",
          "dt_bias": "dt_bias", "norm": "norm", "conv": "conv"}
     t.update(tensors or {})
     self.tensors = t
     H, G = num_heads, num_kv_heads
     # rows of the fused projection: the two low-rank inputs first (so that they start on 16-byte boundaries and the
-    # products behind them can read them in place), then what the convolution runs over, then beta's logits
-    self.a1_off, self.g1_off = 0, decay_rank
-    self.conv_off = decay_rank + gate_rank
+    # products behind them can read them in place) - a gate without a low rank in their place -, then what the
+    # convolution runs over, then beta's logits and a decay's logit a head
+    self.a1_off, self.g1_off = 0, decay_rank or 0
+    self.conv_off = self.g1_off + (gate_rank if gate_rank is not None else H * vdim)
     self.q_off, self.k_off, self.v_off = 0, G * dim, 2 * G * dim      # within the convolved channels
     self.channels = 2 * G * dim + H * vdim
     self.b_off = self.conv_off + self.channels
-    self.proj_width = self.b_off + H
+    self.a_off = self.b_off + H
+    self.proj_width = self.a_off + (H if decay_rank is None else 0)
+    self.proj_width = -(-self.proj_width // 8) * 8      # the rest of the rows is zero
     self.conv_floats = (taps - 1) * self.channels
 
   def cache_spec(self) -> Optional[CacheSpec]:
@@ -137,21 +148,27 @@ class GatedDeltaMixer(Mixer):
   def param_specs(self) -> Dict[str, ParamSpec]:
     W, H, G, D, Dv, K, n, t = self.hidden_size, self.num_heads, self.num_kv_heads, self.dim, self.vdim, self.taps, self.name, self.tensors
     c = t["conv"]
-    return {
+    head_decay, full_gate = self.decay_rank is None, self.gate_rank is None
+    decays = H if head_decay else H * D
+    specs = {
       "proj": ParamSpec((self.proj_width, W), "matrix", [[
         Piece(f"{n}.{t['q']}", self.conv_off + self.q_off, (G * D, W)), Piece(f"{n}.{t['k']}", self.conv_off + self.k_off, (G * D, W)),
         Piece(f"{n}.{t['v']}", self.conv_off + self.v_off, (H * Dv, W)), Piece(f"{n}.{t['b']}", self.b_off, (H, W)),
-        Piece(f"{n}.{t['a1']}", self.a1_off, (self.decay_rank, W)), Piece(f"{n}.{t['g1']}", self.g1_off, (self.gate_rank, W))]]),
+        Piece(f"{n}.{t['a']}", self.a_off, (H, W)) if head_decay else Piece(f"{n}.{t['a1']}", self.a1_off, (self.decay_rank, W)),
+        Piece(f"{n}.{t['g']}", self.g1_off, (H * Dv, W)) if full_gate else Piece(f"{n}.{t['g1']}", self.g1_off, (self.gate_rank, W))]]),
       "conv": ParamSpec((self.channels, K), "vector", [[
         Piece(f"{n}.{t['q']}.{c}", self.q_off, (G * D, K)), Piece(f"{n}.{t['k']}.{c}", self.k_off, (G * D, K)),
         Piece(f"{n}.{t['v']}.{c}", self.v_off, (H * Dv, K))]], init="half_noise"),
-      "a2": ParamSpec((H * D, self.decay_rank), "matrix", [whole(f"{n}.{t['a2']}", (H * D, self.decay_rank))]),
-      "g2": ParamSpec((H * Dv, self.gate_rank), "matrix", [whole(f"{n}.{t['g2']}", (H * Dv, self.gate_rank))]),
-      "dt_bias": ParamSpec((H * D,), "vector", [whole(f"{n}.{t['dt_bias']}", (H * D,))]),
+      "dt_bias": ParamSpec((decays,), "vector", [whole(f"{n}.{t['dt_bias']}", (decays,))]),
       "A_log": ParamSpec((H,), "vector", [whole(f"{n}.{t['A_log']}", (H,))]),
       "norm": ParamSpec((Dv,), "vector", [whole(f"{n}.{t['norm']}", (Dv,))], init="ones_noise"),
       "w_o": ParamSpec((W, H * Dv), "matrix", [whole(f"{n}.{t['o']}", (W, H * Dv))]),
     }
+    if not head_decay:
+      specs["a2"] = ParamSpec((H * D, self.decay_rank), "matrix", [whole(f"{n}.{t['a2']}", (H * D, self.decay_rank))])
+    if not full_gate:
+      specs["g2"] = ParamSpec((H * Dv, self.gate_rank), "matrix", [whole(f"{n}.{t['g2']}", (H * Dv, self.gate_rank))])
+    return specs
 
   def validate(self, dtype: torch.dtype) -> None:
     if self.taps > 16:
@@ -167,14 +184,20 @@ class GatedDeltaMixer(Mixer):
     ops.linear(proj, x, self.proj)
     qkv = ctx.ws.buffer("delta_qkv", (T, self.channels), ctx.dtype)
     ops.causal_conv(qkv, proj[:, self.conv_off:self.conv_off + self.channels], self.conv, None, state[:, :max(self.conv_floats, 1)], ctx, silu=True)
-    decay = ctx.ws.buffer("delta_decay", (T, H * D), ctx.dtype)
-    ops.linear(decay, proj[:, self.a1_off:self.a1_off + self.decay_rank], self.a2)
-    gate = ctx.ws.buffer("delta_gate", (T, H * Dv), ctx.dtype)
-    ops.linear(gate, proj[:, self.g1_off:self.g1_off + self.gate_rank], self.g2)
+    if self.decay_rank is None:
+      decay = proj[:, self.a_off:self.a_off + H]
+    else:
+      decay = ctx.ws.buffer("delta_decay", (T, H * D), ctx.dtype)
+      ops.linear(decay, proj[:, self.a1_off:self.a1_off + self.decay_rank], self.a2)
+    if self.gate_rank is None:
+      gate = proj[:, self.g1_off:self.g1_off + H * Dv]
+    else:
+      gate = ctx.ws.buffer("delta_gate", (T, H * Dv), ctx.dtype)
+      ops.linear(gate, proj[:, self.g1_off:self.g1_off + self.gate_rank], self.g2)
     heads = ctx.ws.buffer("delta_heads", (T, H * Dv), ctx.dtype)
     ops.gated_delta(heads, qkv[:, self.q_off:self.q_off + G * D], qkv[:, self.k_off:self.k_off + G * D], qkv[:, self.v_off:],
                     decay, proj[:, self.b_off:self.b_off + H], gate, self.dt_bias, self.A_log, self.norm, self.norm_eps,
-                    state[:, self.conv_floats:], ctx, H, G, D, Dv, workspace=ctx.ws)
+                    state[:, self.conv_floats:], ctx, H, G, D, Dv, workspace=ctx.ws, gate_silu=self.gate_silu)
     out = ctx.ws.buffer(self.out_buffer, (T, self.hidden_size), ctx.dtype)
     ops.linear(out, heads, self.w_o)
     return out

@@ -170,6 +170,8 @@ def _glu(g, u, glu, limit):
   if glu == "clamped":
     g, u = torch.clamp(g, max=limit), torch.clamp(u, -limit, limit)
     return g * torch.sigmoid(1.702 * g) * (u + 1.0)
+  if glu == "gelu_tanh":
+    return 0.5 * g * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (g + 0.044715 * g ** 3))) * u
   return g * torch.sigmoid(g) * u
 
 
@@ -360,7 +362,7 @@ def rms_pair_sum(out, a, b, w1, w2, eps, scale):
   out.copy_((scale * (w1 * unit(a) + w2 * unit(b))).to(out.dtype))
 
 
-def linear_batched(out, x, w, bias=None, softplus=False, row_gate=None):
+def linear_batched(out, x, w, bias=None, softplus=False, row_gate=None, value_gate=None):
   y = torch.einsum("mbk,bnk->mbn", x.float(), w.float())
   if bias is not None:
     y = y + bias
@@ -368,6 +370,8 @@ def linear_batched(out, x, w, bias=None, softplus=False, row_gate=None):
     y = torch.nn.functional.softplus(y)
   if row_gate is not None:
     y = y * torch.sigmoid(row_gate.float()[:, :x.shape[1], None])
+  if value_gate is not None:
+    y = y * torch.sigmoid(value_gate.float().reshape(y.shape))
   out.copy_(y.to(out.dtype))
 
 
@@ -410,7 +414,8 @@ def selective_scan(y, u, dt_in, bc, b_off, c_off, z, dt_bias, A_log, D, state, c
     state[slot, :inner * N] = S.reshape(-1)
 
 
-def gated_delta(out, q, k, v, a, b, gate, dt_bias, A_log, norm_w, eps, state, ctx, heads, kv_heads, dim, vdim, workspace=None):
+def gated_delta(out, q, k, v, a, b, gate, dt_bias, A_log, norm_w, eps, state, ctx, heads, kv_heads, dim, vdim, workspace=None,
+                gate_silu=False):
   H, G, D, Dv = heads, kv_heads, dim, vdim
   for row0, n, slot in _items(ctx):
     S = state[slot, :H * D * Dv].view(H, D, Dv).clone()
@@ -419,13 +424,14 @@ def gated_delta(out, q, k, v, a, b, gate, dt_bias, A_log, norm_w, eps, state, ct
       qt = qt / torch.sqrt(qt.pow(2).sum(-1, keepdim=True) + 1e-6) * D ** -0.5
       kt = kt / torch.sqrt(kt.pow(2).sum(-1, keepdim=True) + 1e-6)
       qt, kt = qt.repeat_interleave(H // G, dim=0), kt.repeat_interleave(H // G, dim=0)        # [H, D]
-      g = torch.exp(-torch.exp(A_log.float())[:, None] * torch.nn.functional.softplus(a[t].float().view(H, D) + dt_bias.view(H, D)))
+      g = torch.exp(-torch.exp(A_log.float())[:, None] * torch.nn.functional.softplus(a[t].float().view(H, -1) + dt_bias.view(H, -1)))
       beta = torch.sigmoid(b[t].float())                                                       # [H]
       S = g[:, :, None] * S
       u = beta[:, None] * (v[t].float().view(H, Dv) - torch.einsum("hdv,hd->hv", S, kt))
       S = S + kt[:, :, None] * u[:, None, :]
       o = torch.einsum("hdv,hd->hv", S, qt)
-      o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * norm_w * torch.sigmoid(gate[t].float().view(H, Dv))
+      z = gate[t].float().view(H, Dv)
+      o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * norm_w * (z * torch.sigmoid(z) if gate_silu else torch.sigmoid(z))
       out[t] = o.reshape(-1).to(out.dtype)
     state[slot, :H * D * Dv] = S.reshape(-1)
 
