@@ -159,7 +159,7 @@ def build_attention(head_dim: int) -> str:
   return build_library(f"attn_hd{head_dim}", ATTENTION_SOURCES, {"MI_HEAD_DIM": str(head_dim)})
 
 
-def build_all(head_dims: Sequence[int] = (16, 32, 48, 64, 80, 128, 256), remove_stale: bool = True) -> List[str]:
+def build_all(head_dims: Sequence[int] = (16, 32, 48, 64, 80, 96, 128, 256), remove_stale: bool = True) -> List[str]:
   """Builds the common library and the attention library of every head size in ``head_dims``.  Libraries
   of other source versions (another hash in the name) and their compiler logs are then removed from the
   build folder, so that it holds one build."""
