@@ -1550,9 +1550,106 @@ def korurax_one(name: str, cfg: dict, size: dict, batch: int, steps: int, warmup
   return out
 
 
+# ---------------------------------------------------------------------------------------------- --compare besolix
+# The Besolix design beside the closest design the engine has, Vugudra (latent attention, windowed attention and a gated delta
+# rule), at equal size: the sizes of the Vugudra comparison.  Besolix's layers go latent attention, windowed attention, gated
+# delta rule, each with the window of that comparison, and again; from the second round on the latent layers read the first
+# one's latents.  Its delta rule has Vugudra's heads and state, with one decay a head where Vugudra's has one a key channel.
+def besolix_configs(size: dict) -> dict:
+  W, H, G, hd, L = size["width"], size["heads"], size["kv_heads"], size["head"], size["layers"]
+  lat, dl, mask = size["latent"], size["delta"], {"size": COMPARE_WINDOW}
+  latent = dict({k: lat[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "q_rank")}, scale=(lat["dim"] + lat["rot_dim"]) ** -0.5,
+                rot={"dims": lat["rot_dim"], "base": 10000.0}, mask=mask)
+  attn = {"heads": H, "kv_heads": G, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "mask": mask,
+          "rot": {"dims": hd, "base": 500000.0, "scaling": {"factor": 8.0}}}
+  delta = {k: dl[k] for k in ("heads", "kv_heads", "dim", "vdim", "conv")}
+  layers = []
+  for i in range(L):
+    kind, m = (("latent_attention", latent), ("attention", attn), ("delta", delta))[i % 3]
+    if kind == "latent_attention" and i > 0:
+      m = dict(m, kv_from=0)
+    layers.append({"type": kind, "mixer": m, "mlp": {"kind": "dense", "ff": size["ff"]}})
+  bes = {"architecture": "Besolix", "vocab": COMPARE_VOCAB, "width": W, "norm": {"eps": 1e-6}, "layers": layers}
+  return {"vugudra": vugudra_configs(size)["vugudra"], "besolix": bes}
+
+
+def _besolix_groups(times: dict) -> dict:
+  """Vugudra's kinds, its attention split into windowed heads and latent rows (the kernels without TMA and tcgen05)."""
+  import re
+  latent = sum(us for n, us in times.items() if re.search(r"decode_split_kernel|decode_merge|attention_prefill_kernel|attention_generic", n))
+  gate = sum(us for n, us in times.items() if "sigmoid_gate" in n)
+  g = _vugudra_groups(times)
+  g.update(windowed_attention=g["attention"] - latent, latent_attention=latent, value_gate=gate, other=g["other"] - gate)
+  return {k: max(v, 1e-9) for k, v in g.items()}
+
+
+def besolix_one(name: str, cfg: dict, size: dict, batch: int, steps: int, warmup: int, pk: dict, kernels: bool) -> dict:
+  """Prefill and decode of one model of the comparison; with ``kernels`` the device time of its kinds of kernels and the
+  rates they reach against the measured peaks (run with dependent launch off, see main)."""
+  if name == "vugudra":
+    return vugudra_one(name, cfg, size, batch, steps, warmup, pk, kernels)
+  import torch
+  W, H, G, hd, L, T = size["width"], size["heads"], size["kv_heads"], size["head"], size["layers"], PREFILL_TOKENS
+  with tempfile.TemporaryDirectory() as d:
+    with open(os.path.join(d, "config.json"), "w") as f:
+      json.dump(cfg, f)
+    engine = build_engine(d, batch)
+    if not kernels:
+      dec = time_decode(engine, batch, steps, warmup)
+      pre = time_prefill(engine)
+      out = {"decode_tok_s": round(dec["tok_s"], 1), "decode_ms": round(dec["ms"], 4), "launches_per_decode_step": int(dec["launches_per_step"]),
+             "prefill_tok_s": round(T / (pre["ms"] * 1e-3), 1), "prefill_ms": round(pre["ms"], 3)}
+    else:
+      dtimes, ptimes, _ = _step_kernel_times(engine, batch)
+      dk, pt = _besolix_groups(dtimes), _besolix_groups(ptimes)
+      lat, dl, win = size["latent"], size["delta"], COMPARE_WINDOW
+      n_lat, n_att, n_del = (L + 2) // 3, (L + 1) // 3, L // 3
+      lH, D, R, Dv, C, Q = (lat[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "q_rank"))
+      dh, dg, dd, dv = (dl[k] for k in ("heads", "kv_heads", "dim", "vdim"))
+      seen, row, keys = sum(min(t + 1, win) for t in range(T)), -(-(C + R) // 16) * 16, min(CONTEXT, win)
+      ch = 2 * dg * dd + dh * dv                                     # the convolved channels
+      att_w = (2 * H + 2 * G) * hd * W
+      lat_w = n_lat * ((Q + lH * Dv) * W + lH * (D + R) * Q + W * lH * Dv) + (C + R) * W
+      delta_w = (ch + 2 * dh * dv + 2 * dh) * W
+      head_w = n_lat * lH * C * (D + Dv)
+      proj_w = n_att * att_w + lat_w + n_del * delta_w + L * 3 * size["ff"] * W
+      # the recurrence: q, k, v, gate, output and two logits a head once (2 bytes); in a decode step every state in and out
+      delta_io, delta_state = n_del * (2 * dg * dd + dh * (3 * dv + 2)) * 2, n_del * dh * dd * dv * 4 * 2
+      conv_io = n_del * 2 * ch * 2
+
+      def rate(us, amount, peak, unit):      # amount in FLOP or bytes
+        v = amount / us / (1e6 if unit == "TFLOP/s" else 1e3)
+        return {"us": round(us, 1), unit: round(v, 1), "frac": round(v / peak, 4)}
+
+      tf, gb = pk["bf16_tflops"], pk["hbm_gbs"]
+      out = {"prefill_windowed_attention": rate(pt["windowed_attention"], n_att * 4.0 * H * hd * seen, tf, "TFLOP/s"),
+             "decode_windowed_attention": rate(dk["windowed_attention"], batch * keys * n_att * 2 * G * hd * 2, gb, "GB/s"),
+             "prefill_latent_attention": rate(pt["latent_attention"], n_lat * 2.0 * lH * (C + R + C) * seen, tf, "TFLOP/s"),
+             "decode_latent_attention": rate(dk["latent_attention"], batch * keys * n_lat * 2 * row * 2, gb, "GB/s"),
+             "decode_head_products": rate(dk["head_products"], 2.0 * head_w, gb, "GB/s"),
+             "prefill_value_gate": rate(pt["value_gate"], T * n_lat * lH * Dv * 2 * 3, gb, "GB/s"),
+             "prefill_delta_rule": rate(pt["delta_rule"], T * delta_io, gb, "GB/s"),
+             "decode_delta_rule": rate(dk["delta_rule"], batch * (delta_io + delta_state), gb, "GB/s"),
+             "prefill_convolution": rate(pt["convolution"], T * conv_io, gb, "GB/s"), "decode_convolution_us": round(dk["convolution"], 1),
+             "prefill_dense_products": rate(pt["dense_products"] + pt["head_products"], 2.0 * T * (proj_w + head_w), tf, "TFLOP/s"),
+             "decode_dense_products": rate(dk["dense_products"], 2.0 * (proj_w + COMPARE_VOCAB * W), gb, "GB/s"),
+             "other_us": {"prefill": round(pt["other"], 1), "decode": round(dk["other"], 1)}}
+
+      def top_of(times):
+        rows = sorted(((us, n) for n, us in times.items() if not n.startswith("Mem")), reverse=True)[:16]
+        return [[round(us, 1), n.replace("(anonymous namespace)::", "")[:70]] for us, n in rows]
+
+      out["top_kernels_us"] = {"prefill": top_of(ptimes), "decode": top_of(dtimes)}
+    engine.stop()
+    del engine
+    gc.collect()
+    torch.cuda.empty_cache()
+  return out
+
+
 def compare_designs(args) -> int:
   """``--compare rikanex`` / ``--compare vugudra``: the design beside the Qwen3 dense decoder at equal sizes (random weights);
-  ``--compare famupel``: the design beside Vugudra, ``--compare luporax`` and ``--compare korurax``: the design beside Rikanex, each the closest of
+  ``--compare famupel`` and ``--compare besolix``: the design beside Vugudra, ``--compare luporax`` and ``--compare korurax``: the design beside Rikanex, each the closest of
   the engine's designs, at equal sizes: prefill of
   one 2048-token prompt and decode steps at ``--batch`` requests with ``--context``-token contexts, and, from a process of
   its own with dependent launch off, what the kinds of kernels of both reach against the measured peaks."""
@@ -1566,8 +1663,9 @@ def compare_designs(args) -> int:
   sizes_of, configs_of, one = {"rikanex": (COMPARE_SIZES, compare_configs, compare_one), "vugudra": (VUGUDRA_SIZES, vugudra_configs, vugudra_one),
                                "famupel": (FAMUPEL_SIZES, famupel_configs, famupel_one),
                                "luporax": (COMPARE_SIZES, luporax_configs, luporax_one),
-                               "korurax": (COMPARE_SIZES, korurax_configs, korurax_one)}[design]
-  beside = {"famupel": "vugudra", "luporax": "rikanex", "korurax": "rikanex"}.get(design, "qwen3")
+                               "korurax": (COMPARE_SIZES, korurax_configs, korurax_one),
+                               "besolix": (VUGUDRA_SIZES, besolix_configs, besolix_one)}[design]
+  beside = {"famupel": "vugudra", "besolix": "vugudra", "luporax": "rikanex", "korurax": "rikanex"}.get(design, "qwen3")
   result = {"compare": f"{design} beside {beside} at equal sizes", "batch": args.batch, "context": CONTEXT, "window": COMPARE_WINDOW,
             "vocab": COMPARE_VOCAB, "prefill_tokens": PREFILL_TOKENS, "steps": args.steps, "warmup": warmup, "dtype": "bf16",
             "data": "synthetic: random weights, uniform random token ids", "peaks": pk["source"], "sizes": {}}
@@ -1606,8 +1704,8 @@ def main() -> int:
   ap.add_argument("--steps", type=int, default=128)
   ap.add_argument("--warmup", type=int, default=8)
   ap.add_argument("--impl", default="ours", choices=["ours", "reference", "reference-child", "kernels-child", "compare-child"])
-  ap.add_argument("--compare", default=None, choices=["rikanex", "vugudra", "famupel", "luporax", "korurax"],
-                  help="time the Rikanex or the Vugudra design beside the Qwen3 dense decoder, the Famupel design beside Vugudra, or the Luporax or the Korurax design beside Rikanex, at equal sizes (--sizes), print one JSON line and exit")
+  ap.add_argument("--compare", default=None, choices=["rikanex", "vugudra", "famupel", "luporax", "korurax", "besolix"],
+                  help="time the Rikanex or the Vugudra design beside the Qwen3 dense decoder, the Famupel or the Besolix design beside Vugudra, or the Luporax or the Korurax design beside Rikanex, at equal sizes (--sizes), print one JSON line and exit")
   ap.add_argument("--sizes", default="s,m,l", help="with --compare: which of the sizes s, m, l (commas between them)")
   ap.add_argument("--batch", type=int, default=8)
   ap.add_argument("--shape", default="0.6b", choices=sorted(SHAPES), help="layer sizes: the default, or another Qwen3 model's")

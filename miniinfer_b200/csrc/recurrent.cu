@@ -12,6 +12,7 @@
 #include <type_traits>
 
 #include "common.cuh"
+#include "delta_chunk.cuh"
 
 namespace {
 
@@ -304,6 +305,7 @@ struct DeltaPrepArgs {
   float* qn; float* kn;                  // [tokens, kv_heads * dim]
   float* g;                              // [tokens, heads * dim], or [tokens, heads] with one decay a head
   float* qk;                             // [tokens, kv_heads]: qh . kh (one decay a head only)
+  float* lg;                             // [tokens, heads]: ln g (one decay a head only)
   int head_decay;
   float* beta;                           // [tokens, heads]
   const T* v; int ldv;                   // values, head h at column h * vdim
@@ -347,7 +349,11 @@ delta_prepare_kernel(DeltaPrepArgs<T> a) {
       const int h = u - a.kv_heads;
       const float neg_rate = -expf(a.A_log[h]);
       if (a.head_decay) {
-        if (lane == 0) a.g[(size_t)t * a.heads + h] = expf(neg_rate * softplus_f(mi::to_float(a.a[(size_t)t * a.lda + h]) + a.dt_bias[h]));
+        if (lane == 0) {
+          const float lg = fmaxf(neg_rate * softplus_f(mi::to_float(a.a[(size_t)t * a.lda + h]) + a.dt_bias[h]), -1e30f);
+          a.lg[(size_t)t * a.heads + h] = lg;
+          a.g[(size_t)t * a.heads + h] = expf(lg);
+        }
       } else for (int i = lane; i < a.dim; i += 32) {
         const float z = mi::to_float(a.a[(size_t)t * a.lda + (size_t)h * a.dim + i]) + a.dt_bias[h * a.dim + i];
         a.g[((size_t)t * a.heads + h) * a.dim + i] = expf(neg_rate * softplus_f(z));
@@ -384,6 +390,7 @@ struct DeltaArgs {
   float* state; long long state_stride;  // [slot][heads][dim][vdim]
   const int* q_start; const int* q_len; const int* seq_slot;
   int heads, kv_heads, dim, vdim, R;
+  int skip_from;                         // > 0: items of at least so many new tokens are somebody else's (MODE 0)
   // stretches side by side (MODE 1, 2)
   float* seg_state;                      // [item, stretch][heads][dim][vdim]: a stretch's end state from a zero start (MODE 1
                                          // writes), then - after the carry kernel - the state it starts from (MODE 2 reads)
@@ -419,6 +426,7 @@ delta_recurrence_kernel(DeltaArgs<T> a) {
   const int kvh = head / (a.heads / a.kv_heads);
   int row0 = a.q_start[item], n_new = a.q_len[item];
   const int slot = a.seq_slot[item];
+  if (MODE == 0 && a.skip_from > 0 && n_new >= a.skip_from) return;
   if (MODE != 0) {
     const int nseg = delta_segments(n_new);
     if (seg >= nseg) return;
@@ -709,12 +717,18 @@ MI_API int mi_selective_scan(void* y, int ldy, const void* u, int ldu, const voi
   return 0;
 }
 
-// scratch: float32 - unit q and k, decays, q . k, beta, values / read-outs, each starting on a 16-byte boundary
+// scratch: float32 - unit q and k, decays, q . k, the decays' logarithms, beta, values / read-outs, each starting on a 16-byte boundary
 MI_API long long mi_gated_delta_scratch_floats(int T, int heads, int kv_heads, int dim, int vdim, int head_decay) {
-  return (long long)T * ((long long)2 * kv_heads * dim + (long long)heads * (head_decay ? 1 : dim) + kv_heads + heads + (long long)heads * vdim) + 5 * 4;
+  return (long long)T * ((long long)2 * kv_heads * dim + (long long)heads * (head_decay ? 2 : dim) + kv_heads + heads + (long long)heads * vdim) + 6 * 4;
 }
 
 MI_API int mi_gated_delta_segments() { return DELTA_SEGMENTS; }
+
+// Floats of scratch of the walk by chunks, or 0 where it does not take the sizes (one decay a head only).
+MI_API long long mi_gated_delta_chunk_floats(int T, int items, int heads, int dim, int vdim) {
+  if (dim > mi::DELTA_CHUNK_MAX_DIM || dim % 4 != 0 || vdim % 4 != 0) return 0;
+  return mi::delta_chunk_scratch_floats(T, items, heads, dim, vdim);
+}
 
 // Blocks that walk one request's tokens in order (heads x groups of value columns): what a long prompt portion keeps
 // busy without stretches side by side.
@@ -733,7 +747,11 @@ MI_API int mi_gated_delta(void* out, int ldo, const void* q, const void* k, int 
                           const void* b_in, int ldb, const void* gate, int ldg, int dtype, const float* dt_bias, const float* A_log,
                           const float* norm_w, float eps, float* state, long long state_stride, const int* q_start, const int* q_len,
                           const int* seq_slot, int T, int items, int heads, int kv_heads, int dim, int vdim, float* scratch,
-                          float* segments, int head_decay, int gate_silu, cudaStream_t stream) {
+                          float* segments, int head_decay, int gate_silu, float* chunks, int chunk_min, cudaStream_t stream) {
+  // chunks: null, or mi_gated_delta_chunk_floats of scratch - then items of at least chunk_min new tokens are walked a chunk of
+  // tokens at a time (bfloat16 with one decay a head; excludes segments), the others token by token
+  MI_REQUIRE(chunks == nullptr || (dtype == MI_BF16 && head_decay && segments == nullptr && chunk_min > 1),
+             "gated_delta: chunks are for bfloat16 activations and one decay a head");
   // head_decay: a_in [T, heads] and dt_bias [heads], one decay a head, instead of [T, heads * dim] and [heads * dim]
   // segments: null, or items * DELTA_SEGMENTS * heads * dim * (vdim + dim) floats of scratch - then the items' tokens run
   // in stretches side by side (bfloat16 only: the sums then depend on where a portion starts; dim up to 256)
@@ -761,7 +779,8 @@ MI_API int mi_gated_delta(void* out, int ldo, const void* q, const void* k, int 
   float* kn = qn + up4((size_t)T * kv_heads * dim);
   float* g = kn + up4((size_t)T * kv_heads * dim);
   float* qk = g + up4((size_t)T * heads * (head_decay ? 1 : dim));
-  float* beta = qk + up4((size_t)T * kv_heads);
+  float* lg = qk + up4((size_t)T * kv_heads);
+  float* beta = lg + (head_decay ? up4((size_t)T * heads) : 0);
   float* raw = beta + up4((size_t)T * heads);
   dim3 pgrid(T, (heads + kv_heads + 3) / 4 > 16 ? 16 : (heads + kv_heads + 3) / 4);
   dim3 ogrid(T, (heads + 3) / 4 > 16 ? 16 : (heads + 3) / 4);
@@ -772,6 +791,8 @@ MI_API int mi_gated_delta(void* out, int ldo, const void* q, const void* k, int 
   do {                                                                                                            \
     DeltaArgs<TT> d;                                                                                              \
     d.raw = raw; d.qn = qn; d.kn = kn; d.g = g; d.beta = beta; d.qk = qk;                                         \
+    d.skip_from = chunks ? chunk_min : 0;                                                                         \
+    if (chunks && items == 1 && T >= chunk_min) break;                                                            \
     d.vec16 = dim % 4 == 0 && vdim % 4 == 0 && cols % 4 == 0;                                                     \
     d.state = state; d.state_stride = state_stride; d.q_start = q_start; d.q_len = q_len; d.seq_slot = seq_slot;  \
     d.heads = heads; d.kv_heads = kv_heads; d.dim = dim; d.vdim = vdim; d.R = R;                                  \
@@ -799,13 +820,17 @@ MI_API int mi_gated_delta(void* out, int ldo, const void* q, const void* k, int 
     DeltaPrepArgs<TT> p;                                                                                          \
     p.q = (const TT*)q; p.k = (const TT*)k; p.ldqk = ldqk; p.a = (const TT*)a_in; p.lda = lda; p.b = (const TT*)b_in; p.ldb = ldb; \
     p.dt_bias = dt_bias; p.A_log = A_log; p.qn = qn; p.kn = kn; p.g = g; p.beta = beta; p.T_ = T; p.heads = heads;  \
-    p.qk = qk; p.head_decay = head_decay;                                                                         \
+    p.qk = qk; p.lg = lg; p.head_decay = head_decay;                                                                         \
     p.kv_heads = kv_heads; p.dim = dim; p.v = (const TT*)v; p.ldv = ldv; p.raw = raw; p.vdim = vdim;                  \
     mi::launch(delta_prepare_kernel<TT>, pgrid, dim3(128), 0, stream, p);                                         \
     if (DK == 16) MI_DELTA(TT, 16);                                                                               \
     else if (DK == 32) MI_DELTA(TT, 32);                                                                          \
     else if (DK == 64) MI_DELTA(TT, 64);                                                                          \
     else MI_DELTA(TT, 128);                                                                                       \
+    if (chunks) {                                                                                                 \
+      mi::DeltaChunkArgs c{qn, kn, lg, beta, raw, state, state_stride, q_start, q_len, seq_slot, items, heads, kv_heads, dim, vdim, chunk_min}; \
+      if (int e = mi::delta_chunk_run(c, T, chunks, stream)) return e;                                            \
+    }                                                                                                             \
     mi::launch(delta_output_kernel<TT>, ogrid, dim3(128), 0, stream, (TT*)out, ldo, (const float*)raw, (const TT*)gate, ldg, norm_w, heads, vdim, eps, gate_silu); \
   } while (0)
   if (dtype == MI_BF16) MI_DELTA_ALL(__nv_bfloat16);

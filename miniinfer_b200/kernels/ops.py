@@ -604,6 +604,7 @@ DELTA_SEGMENTED_MAX_ITEMS = 4      # the same bound for the delta rule, whose sc
 # B200, 2048 tokens of one request, heads of 128 x 128: 8 heads (64 blocks in order) 5.18 -> 4.57 ms a step of six layers,
 # 16 heads (128 blocks) 7.23 -> 8.11 ms
 DELTA_SEGMENTED_MAX_BLOCKS = 96
+DELTA_CHUNK_MIN_TOKENS = 64        # new tokens a request from which a bfloat16 delta rule with one decay a head goes a chunk at a time
 
 
 def selective_scan(y: torch.Tensor, u: torch.Tensor, dt_in: torch.Tensor, bc: torch.Tensor, b_off: int, c_off: int, z: torch.Tensor,
@@ -670,9 +671,18 @@ def gated_delta(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Te
   n = int(lib.mi_gated_delta_scratch_floats(T, heads, kv_heads, dim, vdim, int(head_decay))) + 8
   scratch = workspace.buffer("gated_delta_scratch", (n,), torch.float32) if workspace is not None else \
     torch.empty(n, dtype=torch.float32, device=v.device)
-  # long prompt portions in bfloat16: each request's tokens in up to 16 stretches side by side (five launches instead of three)
-  segments, launches = None, 3
-  if (v.dtype == torch.bfloat16 and ctx.num_items <= DELTA_SEGMENTED_MAX_ITEMS and T >= SCAN_SEGMENTED_MIN_TOKENS * ctx.num_items
+  # long prompt portions in bfloat16: with one decay a head a chunk of tokens at a time (csrc/delta_chunk.cu); with one a key
+  # channel, or heads too wide for that, each request's tokens in up to 16 stretches side by side (five launches instead of three)
+  segments, chunks, launches = None, None, 3
+  lib.mi_gated_delta_chunk_floats.restype = ctypes.c_longlong
+  if (head_decay and v.dtype == torch.bfloat16 and T - ctx.num_items + 1 >= DELTA_CHUNK_MIN_TOKENS
+      and os.environ.get("MINIINFER_B200_DELTA_CHUNKS", "1") != "0"):
+    m = int(lib.mi_gated_delta_chunk_floats(T, ctx.num_items, heads, dim, vdim))
+    if m > 0:
+      chunks = workspace.buffer("gated_delta_chunks", (m,), torch.float32) if workspace is not None else \
+        torch.empty(m, dtype=torch.float32, device=v.device)
+      launches = 6 if ctx.num_items > 1 else 5
+  if (chunks is None and v.dtype == torch.bfloat16 and ctx.num_items <= DELTA_SEGMENTED_MAX_ITEMS and T >= SCAN_SEGMENTED_MIN_TOKENS * ctx.num_items
       and dim <= 256 and ctx.num_items * int(lib.mi_gated_delta_blocks(heads, dim, vdim)) <= DELTA_SEGMENTED_MAX_BLOCKS
       and os.environ.get("MINIINFER_B200_DELTA_SEGMENTS", "1") != "0"):
     m = ctx.num_items * int(lib.mi_gated_delta_segments()) * heads * dim * (vdim + dim)
@@ -684,7 +694,8 @@ def gated_delta(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Te
                                  ctypes.c_void_p(state.data_ptr()), ctypes.c_longlong(state.stride(0)), _ptr(ctx.q_start, torch.int32),
                                  _ptr(ctx.q_len, torch.int32), _ptr(ctx.seq_slot, torch.int32), T, ctx.num_items, heads, kv_heads, dim, vdim,
                                  _ptr(scratch, torch.float32), _ptr(segments, torch.float32) if segments is not None else _ptr(None),
-                                 int(head_decay), int(gate_silu), _stream()), kernels=launches)
+                                 int(head_decay), int(gate_silu), _ptr(chunks, torch.float32) if chunks is not None else _ptr(None),
+                                 DELTA_CHUNK_MIN_TOKENS, _stream()), kernels=launches)
 
 
 LINEAR_SEGMENTED_MAX_ITEMS = 8     # steps of at most this many requests run long bfloat16 portions in stretches side by side
