@@ -130,6 +130,48 @@ gemm_batched_few_rows_kernel(BatchedArgs a) {
   }
 }
 
+// The same on the tensor cores (mma.sync), where the values of k can be fetched in pairs: a warp takes eight output columns
+// of a batch and the whole of K, straight from global memory, so all of its loads are in flight together.
+__device__ __forceinline__ uint32_t pair_at(const __nv_bfloat16* p, bool take) { return take ? *reinterpret_cast<const uint32_t*>(p) : 0u; }
+
+template <typename TO>
+__global__ void __launch_bounds__(128)
+gemm_batched_mma_few_rows_kernel(BatchedArgs a) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int g = lane >> 2, q = (lane & 3) * 2;
+  const int n0 = (blockIdx.x * 4 + warp) * 8;
+  const int b = blockIdx.y;
+  mi::grid_dependency_sync();
+  if (n0 >= a.N) return;
+  const __nv_bfloat16* x = (const __nv_bfloat16*)a.x + (size_t)b * a.x_batch;
+  const __nv_bfloat16* w = (const __nv_bfloat16*)a.w + (size_t)b * a.w_batch + (size_t)min(n0 + g, a.N - 1) * a.ldw;
+  const bool lo = g < a.M, hi = g + 8 < a.M;
+  const __nv_bfloat16* x0 = x + (size_t)(lo ? g : 0) * a.lda;
+  const __nv_bfloat16* x1 = x + (size_t)(hi ? g + 8 : 0) * a.lda;
+  float c[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 8
+  for (int k = 0; k < a.K; k += 16) {
+    const int ka = k + q, kb = ka + 8;
+    const bool ia = ka < a.K, ib = kb < a.K;
+    const uint32_t w0 = pair_at(w + ka, ia), w1 = pair_at(w + kb, ib);
+    const uint32_t a0 = pair_at(x0 + ka, ia && lo), a1 = pair_at(x1 + ka, ia && hi), a2 = pair_at(x0 + kb, ib && lo), a3 = pair_at(x1 + kb, ib && hi);
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(w0), "r"(w1));
+  }
+  TO* out = (TO*)a.out + (size_t)b * a.o_batch;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int m = g + (i >> 1) * 8, n = n0 + q + (i & 1);
+    if (m >= a.M || n >= a.N) continue;
+    float y = c[i];
+    if (a.bias) y += a.bias[n];
+    if (a.act == 1) y = y > 20.f ? y : log1pf(expf(y));
+    if (a.row_gate) y *= 1.f / (1.f + expf(-__bfloat162float(((const __nv_bfloat16*)a.row_gate)[(size_t)m * a.gate_stride + b])));
+    if (a.value_gate) y *= 1.f / (1.f + expf(-__bfloat162float(((const __nv_bfloat16*)a.value_gate)[(size_t)m * a.gate_stride + (size_t)b * a.N + n])));
+    out[(size_t)m * a.ldo + n] = mi::from_float<TO>(y);
+  }
+}
+
 }  // namespace
 
 MI_API int mi_gemm_batched_few_rows(void* out, int out_dtype, const void* x, const void* w, int dtype, int batch, int M, int N, int K,
@@ -142,6 +184,14 @@ MI_API int mi_gemm_batched_few_rows(void* out, int out_dtype, const void* x, con
   a.x = x; a.w = w; a.out = out; a.x_batch = x_batch; a.w_batch = w_batch; a.o_batch = o_batch;
   a.lda = lda; a.ldw = ldw; a.ldo = ldo; a.M = M; a.N = N; a.K = K; a.bias = bias; a.act = act;
   a.row_gate = row_gate; a.gate_stride = gate_stride; a.value_gate = value_gate;
+  const bool pairs = K % 2 == 0 && lda % 2 == 0 && ldw % 2 == 0 && x_batch % 2 == 0 && w_batch % 2 == 0 && ((uintptr_t)x % 4) == 0 && ((uintptr_t)w % 4) == 0;
+  if (pairs && (out_dtype == MI_BF16 || out_dtype == MI_F32)) {
+    const dim3 mgrid((N + 31) / 32, batch);
+    if (out_dtype == MI_BF16) mi::launch(gemm_batched_mma_few_rows_kernel<__nv_bfloat16>, mgrid, dim3(128), 0, stream, a);
+    else mi::launch(gemm_batched_mma_few_rows_kernel<float>, mgrid, dim3(128), 0, stream, a);
+    MI_LAUNCH_OK("gemm_batched_few_rows");
+    return 0;
+  }
   dim3 grid((N + 3) / 4, batch);
   if (out_dtype == MI_BF16) mi::launch(gemm_batched_few_rows_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, a);
   else if (out_dtype == MI_F32) mi::launch(gemm_batched_few_rows_kernel<float>, grid, dim3(128), 0, stream, a);

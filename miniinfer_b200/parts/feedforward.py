@@ -44,7 +44,7 @@ class SwiGLUFeedForward(FeedForward):
     }
 
   def validate(self, dtype: torch.dtype) -> None:
-    if dtype == torch.bfloat16:
+    if dtype == torch.bfloat16 and self.activation == "silu":      # (the other activations' products take any size)
       for what, k in (("hidden_size", self.hidden_size), ("intermediate_size", self.intermediate_size)):
         if k % 8:
           raise ValueError(f"{self.name}: {what}={k} must be a multiple of 8 in bfloat16 (rows are read 16 bytes at a time)")

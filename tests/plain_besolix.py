@@ -319,6 +319,7 @@ def model(vocab, width, eps, *layers) -> dict:
 # 72, a vocabulary of 333, sixteen query heads on one key/value head, a delta rule of 40 x 8 behind two taps, latent rows of
 # more than 256 values, an eps of 1e-3, a reader that stands behind another latent layer.  E: three latent layers in a row over
 # one cache - nine heads, windows of 200, 64 and 130 -, a delta rule of 48 x 80 with six heads on two behind six taps.
+# F: no size is a multiple of 8, and few are even.
 CONFIGS = {
   "A": model(300, 64, 1e-5,
              latent(3, 24, 8, 16, 24, 40, 24, 10000.0, 0.2, 40),
@@ -352,6 +353,12 @@ CONFIGS = {
              latent(9, 16, 16, 24, 24, 112, 64, 8000.0, 0.2, None, kv_from=0),
              latent(2, 32, 16, 48, 40, 112, 130, 8000.0, 0.15, 32, kv_from=0),
              delta(6, 2, 48, 80, 6, 64)),
+  "F": model(101, 37, 1e-4,
+             latent(3, 9, 6, 5, 11, 21, 13, 400.0, 0.3, 27),
+             delta(3, 3, 7, 9, 3, 18),
+             attention(3, 1, 11, 7, 10, 6, 60.0, 3.0, 0.3, None),
+             latent(1, 5, 6, 13, 7, 21, 6, 400.0, 0.35, 35, kv_from=0),
+             delta(5, 1, 10, 3, 2, None)),
 }
 
 

@@ -229,7 +229,7 @@ def test_a_mistake_in_one_mechanism_would_show(k):
   assert float((diff > 20 * bound).float().mean()) > (0.02 if edge else 0.3), (what, float(diff.max()), bound)
 
 
-@pytest.mark.parametrize("tag,page", [("A", 16), ("B", 8), ("C", 64), ("D", 16), ("E", 64)])
+@pytest.mark.parametrize("tag,page", [("A", 16), ("B", 8), ("C", 64), ("D", 16), ("E", 64), ("F", 8)])
 def test_every_cut_gives_the_plain_logits_on_the_host_path(cpu_kernels, tmp_path, tag, page):
   from miniinfer_b200.engine.replay import TraceRunner
   cfg = plain.CONFIGS[tag]

@@ -17,8 +17,8 @@ from gpu_helpers import DEV
 pytestmark = pytest.mark.gpu
 
 LENGTHS = {"A": (5, 17, 33, 100, 64, 128, 41, 65, 1, 2), "B": (1, 9, 40, 71, 130, 65, 200, 2), "C": (130, 70, 300, 64, 200, 65, 257, 1),
-           "D": (3, 50, 129, 70, 1, 16), "E": (300, 131, 201, 64, 1, 270)}
-PAGES = {"A": 16, "B": 16, "C": 64, "D": 16, "E": 64}
+           "D": (3, 50, 129, 70, 1, 16), "E": (300, 131, 201, 64, 1, 270), "F": (1, 30, 90, 17, 2, 65)}
+PAGES = {"A": 16, "B": 16, "C": 64, "D": 16, "E": 64, "F": 8}
 # bfloat16, as fractions of the root mean square of the plain logits: rounding every product to bfloat16 moves a row by a
 # few hundredths of that, and a first token, whose short row the delta rule's unit norms blow up, by more; a wrong key, a
 # window's edge one off or a lost state moves most rows by tenths, and shows in the float32 runs, which take the same path
@@ -74,7 +74,7 @@ def compare(got, ref, dtype, what):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("tag", ["A", "B", "C", "D", "E"])
+@pytest.mark.parametrize("tag", ["A", "B", "C", "D", "E", "F"])
 @pytest.mark.parametrize("cut", ["whole", "tail", "portions", "mixed", "preempted"])
 def test_every_cut_gives_the_plain_logits(besolix_dirs, dtype, tag, cut):
   d = besolix_dirs(tag)
