@@ -507,7 +507,7 @@ def kernel_case(name: str, reps: int = 3) -> str:
     out = torch.empty(T, W, dtype=torch.bfloat16, device=dev)
     fn = lambda: ops.routed_experts(out, x, router, corr, gate_up, down, top, ws)
     what = f"{T} tokens, {E} experts of 3 x {F} x {W}, {top} a token ({T * top * 3 * 2 * F * W / 1e9:.1f} GFLOP)"
-  elif name in ("selective_scan", "delta_rule"):
+  elif name in ("selective_scan", "delta_rule", "delta_rule_head_decay"):
     # one prompt portion of 8192 tokens (a recurrence walks it in order) beside seven decode tokens of other requests
     from types import SimpleNamespace
     cuts = [8192] + [1] * 7
@@ -526,8 +526,9 @@ def kernel_case(name: str, reps: int = 3) -> str:
     else:
       H, G, Dk, Dv = 16, 8, 128, 128
       q, k, v = rnd(T, G * Dk), rnd(T, G * Dk), rnd(T, H * Dv)
-      a_in, b_in, gate = rnd(T, H * Dk), rnd(T, H), rnd(T, H * Dv)
-      dt_bias, A_log, norm_w = rnd(H * Dk, dtype=torch.float32) - 1.0, rnd(H, dtype=torch.float32) * 0.3, 1 + 0.1 * rnd(Dv, dtype=torch.float32)
+      decays = H if name == "delta_rule_head_decay" else H * Dk
+      a_in, b_in, gate = rnd(T, decays), rnd(T, H), rnd(T, H * Dv)
+      dt_bias, A_log, norm_w = rnd(decays, dtype=torch.float32) - 1.0, rnd(H, dtype=torch.float32) * 0.3, 1 + 0.1 * rnd(Dv, dtype=torch.float32)
       state = torch.zeros((len(cuts), H * Dk * Dv), dtype=torch.float32, device=dev)
       out = torch.empty(T, H * Dv, dtype=torch.bfloat16, device=dev)
       fn = lambda: ops.gated_delta(out, q, k, v, a_in, b_in, gate, dt_bias, A_log, norm_w, 1e-6, state, ctx, H, G, Dk, Dv, workspace=ws)
@@ -594,7 +595,7 @@ def kernel_case(name: str, reps: int = 3) -> str:
 
 KERNEL_CASES = ("sample", "silu_mul", "gemm_f32", "gemm_tc_plain", "gemm_stream", "attention_generic", "attention_prefill_tc",
                 "attention_prefill_tc_pairs", "attention_prefill_mma", "attention_decode_cpasync", "experts_many_rows", "experts_few_rows",
-                "selective_scan", "delta_rule", "linear_attention", "hyper_connection", "attention_prefill_tc_sigmoid", "attention_decode_tma_sigmoid",
+                "selective_scan", "delta_rule", "delta_rule_head_decay", "linear_attention", "hyper_connection", "attention_prefill_tc_sigmoid", "attention_decode_tma_sigmoid",
                 "rglru_recurrence", "mingru_recurrence", "attention_prefill_tc_distance", "attention_prefill_latent", "residual_step")
 
 
@@ -955,7 +956,8 @@ def _vugudra_groups(times: dict) -> dict:
       g["head_products"] += us
     elif "selective_scan" in name or "scan_carry" in name:
       g["scan"] += us
-    elif "gated_delta" in name or "delta_recurrence" in name or "delta_prepare" in name or "delta_output" in name or "delta_carry" in name:
+    elif "gated_delta" in name or "delta_recurrence" in name or "delta_prepare" in name or "delta_output" in name or "delta_carry" in name or \
+        re.search(r"chunk_(solve|state|out)_kernel", name):
       g["delta_rule"] += us
     elif "causal_conv" in name or "conv_state" in name:
       g["convolution"] += us

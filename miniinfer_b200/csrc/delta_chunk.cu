@@ -87,12 +87,14 @@ chunk_solve_kernel(Args a) {
   const int first = found[1] * C, n = min(C, a.q_len[item] - first), row0 = a.q_start[item] + first;
   const int kvh = head / (a.heads / a.kv_heads);
   const size_t unit = (size_t)blockIdx.x * a.heads + head;
-  for (int i = tid; i < C * (a.dp / 4); i += THREADS) {
-    const int t = i / (a.dp / 4), d = (i - t * (a.dp / 4)) * 4;
-    const bool in = t < n && d < a.dim;
-    const size_t from = in ? ((size_t)(row0 + t) * a.kv_heads + kvh) * a.dim + d : 0;
-    copy16(ks + t * ld + d, a.kn + from, in);
-    copy16(qs + t * ld + d, a.qn + from, in);
+  {
+    const int per_row = a.dp / 4, rows = THREADS / per_row, t0 = tid / per_row, d = (tid - t0 * per_row) * 4;
+    for (int t = t0; t < C && t0 < rows; t += rows) {
+      const bool in = t < n && d < a.dim;
+      const size_t from = in ? ((size_t)(row0 + t) * a.kv_heads + kvh) * a.dim + d : 0;
+      copy16(ks + t * ld + d, a.kn + from, in);
+      copy16(qs + t * ld + d, a.qn + from, in);
+    }
   }
   copies_begun();
   if (tid < 32) {                      // two tokens a lane (tokens behind the last: no decay, nothing written)
@@ -215,18 +217,24 @@ chunk_state_kernel(Args a) {
   float* bufs = sm;                    // two of: W^T [dp][C], K [C][dp], U0 [C][CB], e^G and e^(G_C - G) [2 C]
   float* S = bufs + 2 * buf_floats;    // [dp][CB]
   float* us = S + dp * CB;             // [C][CB] e^(G_C - G) U
-  float* part = us + C * CB;           // [8][C][CB]
+  float* part = us + C * CB;           // [8][C][CB], a token's row at place t ^ ((t >> 2) & 1)
   mi::grid_dependency_sync();
+  // which of K's 16-byte pieces this thread copies: one of a row, of every `rows`-th row
+  const int per_row = dp / 4, rows = THREADS / per_row, kt = tid / per_row, kd = (tid - kt * per_row) * 4;
   auto fetch = [&](int c, float* buf) {
     const size_t unit = (size_t)(c - a.c0) * a.heads + head;
     const int first = (c - base) * C, n = min(C, n_new - first);
     const float* w = a.wt + unit * dp * C;
     for (int i = tid; i < dp * C / 4; i += THREADS) copy16(buf + 4 * i, w + 4 * i, true);
     float* kb = buf + dp * C;
-    for (int i = tid; i < C * (dp / 4); i += THREADS) {
-      const int t = i / (dp / 4), d = (i - t * (dp / 4)) * 4;
-      const bool in = t < n && d < a.dim;
-      copy16(kb + t * dp + d, a.kn + (in ? ((size_t)(row0 + first + t) * a.kv_heads + kvh) * a.dim + d : 0), in);
+    if (kt < rows) {
+      const size_t step = (size_t)a.kv_heads * a.dim;
+      const float* k = a.kn + (size_t)(row0 + first) * step + (size_t)kvh * a.dim + kd;
+#pragma unroll 8
+      for (int t = kt; t < C; t += rows) {
+        const bool in = t < n && kd < a.dim;
+        copy16(kb + t * dp + kd, in ? k + t * step : a.kn, in);
+      }
     }
     float* ub = kb + C * dp;
     copy16(ub + 4 * tid, a.u + unit * C * a.vp + (size_t)(tid / 4) * a.vp + v0 + (tid % 4) * 4, true);      // C * CB / 4 = THREADS
@@ -284,7 +292,7 @@ chunk_state_kernel(Args a) {
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
         const int t = (i < 4 ? 0 : 28) + rg * 4 + i;
-        st4(part + ((size_t)warp * C + t) * CB + cg, make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]));
+        st4(part + ((size_t)warp * C + (t ^ (rg & 1))) * CB + cg, make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]));
       }
     }
     __syncthreads();
@@ -293,7 +301,7 @@ chunk_state_kernel(Args a) {
       float4 x = ld4(ub + t * CB + cg);
 #pragma unroll
       for (int k = 0; k < 8; ++k) {
-        const float4 y = ld4(part + ((size_t)k * C + t) * CB + cg);
+        const float4 y = ld4(part + ((size_t)k * C + (t ^ ((t >> 2) & 1))) * CB + cg);
         x.x -= y.x; x.y -= y.y; x.z -= y.z; x.w -= y.w;
       }
       st4(a.u + unit * C * a.vp + (size_t)t * a.vp + v0 + cg, x);
@@ -418,6 +426,8 @@ long long delta_chunk_scratch_floats(int T, int items, int heads, int dim, int v
   const long long chunks = most_chunks(T, items) < slab_chunks(heads) ? most_chunks(T, items) : slab_chunks(heads);
   return chunks * heads * unit_floats(pad(dim, 32), pad(vdim, CB));
 }
+
+int delta_chunk_slabs(int T, int items, int heads) { return (most_chunks(T, items) + slab_chunks(heads) - 1) / slab_chunks(heads); }
 
 int delta_chunk_run(const DeltaChunkArgs& in, int T, float* scratch, cudaStream_t stream) {
   MI_REQUIRE(in.dim > 0 && in.dim <= DELTA_CHUNK_MAX_DIM && in.dim % 4 == 0 && in.vdim % 4 == 0 && in.min_tokens > 0,

@@ -20,6 +20,7 @@ struct DeltaChunkArgs {
 
 // Floats of scratch for a step of T tokens in `items` items (some slabs of chunks at a time share it).
 long long delta_chunk_scratch_floats(int T, int items, int heads, int dim, int vdim);
+int delta_chunk_slabs(int T, int items, int heads);      // three launches each
 int delta_chunk_run(const DeltaChunkArgs& a, int T, float* scratch, cudaStream_t stream);
 
 }  // namespace mi

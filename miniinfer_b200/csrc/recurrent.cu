@@ -730,6 +730,8 @@ MI_API long long mi_gated_delta_chunk_floats(int T, int items, int heads, int di
   return mi::delta_chunk_scratch_floats(T, items, heads, dim, vdim);
 }
 
+MI_API int mi_gated_delta_chunk_slabs(int T, int items, int heads) { return mi::delta_chunk_slabs(T, items, heads); }
+
 // Blocks that walk one request's tokens in order (heads x groups of value columns): what a long prompt portion keeps
 // busy without stretches side by side.
 MI_API int mi_gated_delta_blocks(int heads, int dim, int vdim) {

@@ -604,7 +604,10 @@ DELTA_SEGMENTED_MAX_ITEMS = 4      # the same bound for the delta rule, whose sc
 # B200, 2048 tokens of one request, heads of 128 x 128: 8 heads (64 blocks in order) 5.18 -> 4.57 ms a step of six layers,
 # 16 heads (128 blocks) 7.23 -> 8.11 ms
 DELTA_SEGMENTED_MAX_BLOCKS = 96
-DELTA_CHUNK_MIN_TOKENS = 64        # new tokens a request from which a bfloat16 delta rule with one decay a head goes a chunk at a time
+# New tokens a request from which a bfloat16 delta rule with one decay a head goes a chunk at a time.  Measured on B200, heads
+# of 128 x 128, the whole operation, chunks / in order in microseconds: 8 heads 78 / 85 at 128 tokens and 85 / 154 at 256; 16
+# heads 96 / 87 and 106 / 155; 32 heads 104 / 89 and 126 / 163
+DELTA_CHUNK_MIN_TOKENS = 160
 
 
 def selective_scan(y: torch.Tensor, u: torch.Tensor, dt_in: torch.Tensor, bc: torch.Tensor, b_off: int, c_off: int, z: torch.Tensor,
@@ -681,7 +684,7 @@ def gated_delta(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Te
     if m > 0:
       chunks = workspace.buffer("gated_delta_chunks", (m,), torch.float32) if workspace is not None else \
         torch.empty(m, dtype=torch.float32, device=v.device)
-      launches = 6 if ctx.num_items > 1 else 5
+      launches = (3 if ctx.num_items > 1 else 2) + 3 * int(lib.mi_gated_delta_chunk_slabs(T, ctx.num_items, heads))
   if (chunks is None and v.dtype == torch.bfloat16 and ctx.num_items <= DELTA_SEGMENTED_MAX_ITEMS and T >= SCAN_SEGMENTED_MIN_TOKENS * ctx.num_items
       and dim <= 256 and ctx.num_items * int(lib.mi_gated_delta_blocks(heads, dim, vdim)) <= DELTA_SEGMENTED_MAX_BLOCKS
       and os.environ.get("MINIINFER_B200_DELTA_SEGMENTS", "1") != "0"):

@@ -119,7 +119,7 @@ def test_delta_rule_of_long_portions(dtype, H, G, D, Dv):
   c = DeltaCase(T, H, G, D, Dv, dtype, shift=-3.0)
   want, last = c.want()
   bound = 2 * tol(dtype) * max(1.0, float(want.abs().max()) / 4)
-  for cuts in ((600, 2, 690, 1, 1, 1, 1, 1, 1, 1, 1), (1290,) + (1,) * 10, (520, 780), (63, 64, 65, 128, 129, 127, 192, 532)):
+  for cuts in ((600, 2, 690, 1, 1, 1, 1, 1, 1, 1, 1), (1290,) + (1,) * 10, (520, 780), (63, 64, 159, 160, 161, 128, 192, 373)):
     for others in ((), ((0, 0, 1), (1, 0, 37), (3, 10, 12))):
       state = torch.zeros((4, H * D * Dv), dtype=torch.float32, device=DEV)
       got, pos = [], 0
