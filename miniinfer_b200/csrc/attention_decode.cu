@@ -394,6 +394,8 @@ decode_split_kernel(DecodeArgs a) {
 // The merge as a kernel of its own, a block per (request, query head): with many query heads on one kv head the block
 // that finishes a request last would have heads x pieces partial rows to add, one after another.  The same algebra as
 // the merge inside decode_split_kernel, pieces in ascending order; which of the two runs depends on the head counts alone.
+constexpr int MERGE_PIECES = 512;
+
 __global__ void __launch_bounds__(128)
 decode_merge_kernel(DecodeArgs a) {
   mi::grid_dependency_sync();
@@ -406,18 +408,30 @@ decode_merge_kernel(DecodeArgs a) {
   const int row = a.q_start[item];
   const float* ml = a.part_ml + ((size_t)e * a.nh + head) * a.max_splits * 2;
   const float* po = a.part_o + ((size_t)e * a.nh + head) * a.max_splits * HD;
+  // the pieces' maxima and sums come together, a thread each; then every thread goes through them in shared memory
+  __shared__ float s_m[MERGE_PIECES], s_l[MERGE_PIECES];
+  const bool here = n_splits <= MERGE_PIECES;
+  if (here) {
+    for (int s = threadIdx.x; s < n_splits; s += blockDim.x) {
+      s_m[s] = ml[2 * s];
+      s_l[s] = ml[2 * s + 1];
+    }
+    __syncthreads();
+  }
+  auto piece_m = [&](int s) { return here ? s_m[s] : ml[2 * s]; };
+  auto piece_l = [&](int s) { return here ? s_l[s] : ml[2 * s + 1]; };
   float m = -INFINITY;
-  for (int s = 0; s < n_splits; ++s) m = fmaxf(m, ml[2 * s]);
+  for (int s = 0; s < n_splits; ++s) m = fmaxf(m, piece_m(s));
   const float sink2 = a.sink ? a.sink[head] * 1.4426950408889634f : -INFINITY;
   m = fmaxf(m, sink2);
   float l = 0.f;
-  for (int s = 0; s < n_splits; ++s) l = fmaf(ml[2 * s + 1], exp2f(ml[2 * s] - m), l);
+  for (int s = 0; s < n_splits; ++s) l = fmaf(piece_l(s), exp2f(piece_m(s) - m), l);
   if (a.sink) l += exp2f(sink2 - m);
   const float inv = a.score_bias ? exp2f(m) : 1.f / l;
   for (int d = threadIdx.x; d < a.out_hd; d += blockDim.x) {
     float acc = 0.f;
 #pragma unroll 8
-    for (int s = 0; s < n_splits; ++s) acc = fmaf(po[(size_t)s * HD + d], exp2f(ml[2 * s] - m), acc);
+    for (int s = 0; s < n_splits; ++s) acc = fmaf(po[(size_t)s * HD + d], exp2f(piece_m(s) - m), acc);
     float y = acc * inv;
     if (a.gate) y = __fdividef(y, 1.f + __expf(-__bfloat162float(a.gate[(size_t)row * a.gate_stride + mi::gate_index(head, d, a.out_hd, a.gate_per_head)])));
     a.out[((size_t)row * a.nh + head) * a.out_hd + d] = __float2bfloat16_rn(y);
