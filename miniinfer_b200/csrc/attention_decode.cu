@@ -396,7 +396,7 @@ decode_split_kernel(DecodeArgs a) {
 // the merge inside decode_split_kernel, pieces in ascending order; which of the two runs depends on the head counts alone.
 constexpr int MERGE_PIECES = 512;
 
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 decode_merge_kernel(DecodeArgs a) {
   mi::grid_dependency_sync();
   const int head = blockIdx.x, e = blockIdx.y;
@@ -408,30 +408,33 @@ decode_merge_kernel(DecodeArgs a) {
   const int row = a.q_start[item];
   const float* ml = a.part_ml + ((size_t)e * a.nh + head) * a.max_splits * 2;
   const float* po = a.part_o + ((size_t)e * a.nh + head) * a.max_splits * HD;
-  // the pieces' maxima and sums come together, a thread each; then every thread goes through them in shared memory
+  // the pieces' maxima, sums and factors are fetched and made a thread each (the first MERGE_PIECES of them) and read from
+  // shared memory by all
   __shared__ float s_m[MERGE_PIECES], s_l[MERGE_PIECES];
-  const bool here = n_splits <= MERGE_PIECES;
-  if (here) {
-    for (int s = threadIdx.x; s < n_splits; s += blockDim.x) {
-      s_m[s] = ml[2 * s];
-      s_l[s] = ml[2 * s + 1];
-    }
-    __syncthreads();
+  const int near = min(n_splits, MERGE_PIECES);
+  for (int s = threadIdx.x; s < near; s += blockDim.x) {
+    s_m[s] = ml[2 * s];
+    s_l[s] = ml[2 * s + 1];
   }
-  auto piece_m = [&](int s) { return here ? s_m[s] : ml[2 * s]; };
-  auto piece_l = [&](int s) { return here ? s_l[s] : ml[2 * s + 1]; };
+  __syncthreads();
   float m = -INFINITY;
-  for (int s = 0; s < n_splits; ++s) m = fmaxf(m, piece_m(s));
+  for (int s = 0; s < near; ++s) m = fmaxf(m, s_m[s]);
+  for (int s = near; s < n_splits; ++s) m = fmaxf(m, ml[2 * s]);
   const float sink2 = a.sink ? a.sink[head] * 1.4426950408889634f : -INFINITY;
   m = fmaxf(m, sink2);
+  __syncthreads();
+  for (int s = threadIdx.x; s < near; s += blockDim.x) s_m[s] = exp2f(s_m[s] - m);
+  __syncthreads();
   float l = 0.f;
-  for (int s = 0; s < n_splits; ++s) l = fmaf(piece_l(s), exp2f(piece_m(s) - m), l);
+  for (int s = 0; s < near; ++s) l = fmaf(s_l[s], s_m[s], l);
+  for (int s = near; s < n_splits; ++s) l = fmaf(ml[2 * s + 1], exp2f(ml[2 * s] - m), l);
   if (a.sink) l += exp2f(sink2 - m);
   const float inv = a.score_bias ? exp2f(m) : 1.f / l;
   for (int d = threadIdx.x; d < a.out_hd; d += blockDim.x) {
     float acc = 0.f;
 #pragma unroll 8
-    for (int s = 0; s < n_splits; ++s) acc = fmaf(po[(size_t)s * HD + d], exp2f(piece_m(s) - m), acc);
+    for (int s = 0; s < near; ++s) acc = fmaf(po[(size_t)s * HD + d], s_m[s], acc);
+    for (int s = near; s < n_splits; ++s) acc = fmaf(po[(size_t)s * HD + d], exp2f(ml[2 * s] - m), acc);
     float y = acc * inv;
     if (a.gate) y = __fdividef(y, 1.f + __expf(-__bfloat162float(a.gate[(size_t)row * a.gate_stride + mi::gate_index(head, d, a.out_hd, a.gate_per_head)])));
     a.out[((size_t)row * a.nh + head) * a.out_hd + d] = __float2bfloat16_rn(y);
@@ -495,7 +498,7 @@ MI_API int mi_attention_decode_bf16(void* out, const void* q_base, int q_stride,
   // more than eight query heads on a kv head: the merge as a kernel of its own, a block per (request, head)
   a.merge_apart = nh / nkv > 8 ? 1 : 0;
   mi::launch(distance ? decode_split_kernel<true> : decode_split_kernel<false>, dim3(dim3(nkv, max_splits, n_dec)), dim3(WARPS * 32), SMEM_BYTES, stream, a);
-  if (a.merge_apart) mi::launch(decode_merge_kernel, dim3(nh, n_dec), dim3(128), 0, stream, a);
+  if (a.merge_apart) mi::launch(decode_merge_kernel, dim3(nh, n_dec), dim3(out_hd > 128 ? 256 : 128), 0, stream, a);
   MI_LAUNCH_OK("attention_decode");
   return 0;
 }
