@@ -326,7 +326,7 @@ def test_latent_attention_with_a_window_a_value_gate_and_a_reader(dtype, H, D, R
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("nh,hd,page,window,ohd", [(3, 48, 16, 24, 40), (8, 96, 64, 70, 64), (9, 128, 64, 64, 112), (16, 256, 64, 100, 192), (2, 272, 16, 33, 264),
+@pytest.mark.parametrize("nh,hd,page,window,ohd", [(3, 48, 16, 24, 40), (7, 96, 64, 70, 80), (9, 128, 64, 64, 112), (16, 256, 64, 100, 192), (2, 272, 16, 33, 264),
                                                    (20, 64, 64, 1, 48)])
 def test_keys_on_both_sides_of_a_windows_edge_in_latent_rows(dtype, nh, hd, page, window, ohd):
   """Many query heads on one key/value head whose output is narrower than its rows: the oldest key a token still sees and the
@@ -357,7 +357,7 @@ def test_keys_on_both_sides_of_a_windows_edge_in_latent_rows(dtype, nh, hd, page
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("H,G,D,Dv,dims,base,factor", [(4, 2, 24, 40, 16, 300.0, 4.0), (3, 3, 32, 16, 32, 90.0, 1.0), (4, 1, 96, 96, 24, 50000.0, 8.0), (2, 1, 8, 8, 2, 10.0, 0.5)])
+@pytest.mark.parametrize("H,G,D,Dv,dims,base,factor", [(4, 2, 24, 40, 16, 300.0, 4.0), (3, 3, 32, 16, 32, 90.0, 1.0), (6, 2, 88, 96, 36, 30000.0, 6.0), (2, 1, 8, 8, 2, 10.0, 0.5)])
 def test_normed_heads_rotated_by_divided_frequencies(dtype, H, G, D, Dv, dims, base, factor):
   from miniinfer_b200.kernels import ops
   from miniinfer_b200.parts import LinearScaledRotaryEncoding
